@@ -44,6 +44,9 @@ struct WinArgs {
     int chunk;              // 0: none
     int max_pages, q_stride, gate_stride, nh, nkvh, dk, dv, hc, splits, window, keep_first;
     float scale, softcap;
+    int gate_per_head = 0;  // 1: the gate holds one number per (token, head)
+    float out_scale = 1.f;  // multiplies the output
+    int ldo = 0;            // row pitch of out (0: nh * dv)
 };
 
 template <typename T, int DPL>
@@ -153,8 +156,8 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(const W
         const int tq = r / nheads, hh = r - tq * nheads;
         const int t = t0 + tq, h = h0 + hh;
         if (a.splits == 1) {
-            T* dst = static_cast<T*>(a.out) + ((size_t)t * a.nh + h) * dv;
-            const T* gt = a.gate ? static_cast<const T*>(a.gate) + (size_t)t * a.gate_stride + (size_t)h * dv : nullptr;
+            T* dst = static_cast<T*>(a.out) + (size_t)t * a.ldo + (size_t)h * dv;
+            const T* gt = a.gate ? static_cast<const T*>(a.gate) + (size_t)t * a.gate_stride + (a.gate_per_head ? (size_t)h : (size_t)h * dv) : nullptr;
             float lsum = l[i], keep = 1.f;
             if (a.sinks) {          // the sink joins the denominator; the larger of it and the maximum stays the reference
                 const float sk = a.sinks[h];
@@ -165,7 +168,8 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(const W
                     lsum += expf(sk - m[i]);
                 }
             }
-            const float inv = keep / lsum;
+            float inv = keep / lsum * a.out_scale;
+            if (gt && a.gate_per_head) inv *= 1.0f / (1.0f + expf(-ldf(gt)));
             const int pos_t = a.ocos ? a.tok_pos[t] : 0;
 #pragma unroll
             for (int c = 0; c < DPL; ++c) {
@@ -180,7 +184,7 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(const W
                     }
                 }
                 if (ch < dv) {
-                    if (gt) v *= 1.0f / (1.0f + expf(-ldf(gt + ch)));
+                    if (gt && !a.gate_per_head) v *= 1.0f / (1.0f + expf(-ldf(gt + ch)));
                     stf(dst + ch, v);
                 }
             }
@@ -204,7 +208,8 @@ template <typename T>
 __global__ void attention_window_merge_kernel(const float* __restrict__ partial, T* __restrict__ out,
                                               const T* __restrict__ gate, int gate_stride, int nh, int dv, int splits,
                                               const float* __restrict__ sinks, const float* __restrict__ ocos,
-                                              const float* __restrict__ osin, const int* __restrict__ tok_pos) {
+                                              const float* __restrict__ osin, const int* __restrict__ tok_pos,
+                                              int gate_per_head, float out_scale, int ldo) {
     pdl_sync();
     const int t = blockIdx.x, h = blockIdx.y;
     const float* p = partial + ((size_t)t * nh + h) * splits * (dv + 2);
@@ -232,8 +237,8 @@ __global__ void attention_window_merge_kernel(const float* __restrict__ partial,
             const float co = ocos[(size_t)tok_pos[t] * (dv / 2) + (c >> 1)], si = osin[(size_t)tok_pos[t] * (dv / 2) + (c >> 1)];
             v = (c & 1) ? v * co - other * si : v * co + other * si;
         }
-        if (gate) v *= 1.0f / (1.0f + expf(-ldf(gate + (size_t)t * gate_stride + (size_t)h * dv + c)));
-        stf(out + ((size_t)t * nh + h) * dv + c, v);
+        if (gate) v *= 1.0f / (1.0f + expf(-ldf(gate + (size_t)t * gate_stride + (gate_per_head ? (size_t)h : (size_t)h * dv + c))));
+        stf(out + (size_t)t * ldo + (size_t)h * dv + c, v * out_scale);
     }
 }
 
@@ -260,6 +265,8 @@ static int window_launch(WinArgs a, int tiles, int nt, cudaStream_t s) {
     if (a.nh <= 0 || a.nkvh <= 0 || a.nh % a.nkvh || a.window <= 0 || a.keep_first < 0) return TB_ERR_ARG;
     if (a.dk <= 0 || a.dv <= 0 || a.dk > 256 || a.dv > 256) return TB_ERR_UNSUPPORTED;
     if (a.splits < 1 || (a.splits > 1 && !a.partial)) return TB_ERR_ARG;
+    if (a.ldo == 0) a.ldo = a.nh * a.dv;
+    if (a.ldo < a.nh * a.dv) return TB_ERR_ARG;
     if (a.chunk < 0 || (a.ocos && (!a.osin || a.dv % 2))) return TB_ERR_ARG;
     if (tiles <= 0 || nt <= 0) return tiles == 0 || nt == 0 ? 0 : TB_ERR_ARG;
     const int group = a.nh / a.nkvh;
@@ -279,7 +286,8 @@ static int window_launch(WinArgs a, int tiles, int nt, cudaStream_t s) {
     if (a.splits > 1) {
         dim3 grid(nt, a.nh);
         TB_LAUNCH((attention_window_merge_kernel<T>), grid, a.dv < 128 ? 64 : 128, 0, s, a.partial, (T*)a.out,
-                  (const T*)a.gate, a.gate_stride, a.nh, a.dv, a.splits, a.sinks, a.ocos, a.osin, a.tok_pos);
+                  (const T*)a.gate, a.gate_stride, a.nh, a.dv, a.splits, a.sinks, a.ocos, a.osin, a.tok_pos, a.gate_per_head,
+                  a.out_scale, a.ldo);
         rc = tb_last_error();
     }
     return rc;
@@ -297,10 +305,27 @@ extern "C" {
                   softcap};                                                                                           \
         return window_launch<T>(a, tiles, nt, s);                                                                     \
     }
+// The same with a gate of one number per (token, head) (gate_per_head), a multiplier of the output and a row pitch of
+// the output, for a mixer whose result lands in a wider row.
+#define TB_ATTENTION_WINDOW_HEADS(NAME, T)                                                                            \
+    int NAME(const void* q, void* out, const void* kc, const void* vc, const void* gate, const int* tile_seq,         \
+             const int* tile_t0, const int* tile_nq, const int* tok_pos, const int* page_table, float* partial,       \
+             int tiles, int nt, int max_pages, int q_stride, int gate_stride, int nh, int nkvh, int dk, int dv,       \
+             int splits, int window, int keep_first, float scale, float softcap, int chunk, const float* sinks,       \
+             const float* ocos, const float* osin, int gate_per_head, float out_scale, int ldo, cudaStream_t s) {     \
+        WinArgs a{q, out, kc, vc, gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, ocos, osin,  \
+                  chunk, max_pages, q_stride, gate_stride, nh, nkvh, dk, dv, 0, splits, window, keep_first, scale,    \
+                  softcap, gate_per_head, out_scale, ldo};                                                            \
+        return window_launch<T>(a, tiles, nt, s);                                                                     \
+    }
+TB_ATTENTION_WINDOW_HEADS(tb_attention_window_heads_f32, float)
+TB_ATTENTION_WINDOW_HEADS(tb_attention_window_heads_bf16, __nv_bfloat16)
 TB_ATTENTION_WINDOW(tb_attention_window_f32, float)
 TB_ATTENTION_WINDOW(tb_attention_window_bf16, __nv_bfloat16)
 }
 
 #include "tape.h"
+TB_TAPE_REGISTER(tb_attention_window_heads_f32)
+TB_TAPE_REGISTER(tb_attention_window_heads_bf16)
 TB_TAPE_REGISTER(tb_attention_window_f32)
 TB_TAPE_REGISTER(tb_attention_window_bf16)

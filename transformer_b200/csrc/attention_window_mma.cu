@@ -43,6 +43,9 @@ struct WinMmaArgs {
     int chunk;                   // > 0: position i sees j only if i / chunk == j / chunk
     int tiles, max_pages, q_stride, gate_stride, nh, nkvh, splits, window, keep_first;
     float scale, softcap;
+    int gate_per_head = 0;  // 1: the gate holds one number per (token, head)
+    float out_scale = 1.f;  // multiplies the output
+    int ldo = 0;            // row pitch of out (0: nh * DV)
 };
 
 __host__ __device__ constexpr int wm_blocks(int dk, int dv) { return (dk + dv) <= 256 ? 3 : 1; }
@@ -257,11 +260,13 @@ __global__ void __launch_bounds__(WM_THREADS, wm_blocks(DK, DV)) attention_windo
                     lsum += exp2f(sk - m_run[r]);
                 }
             }
-            const float inv = keep / lsum;
+            float inv = keep / lsum * a.out_scale;
+            if (a.gate && a.gate_per_head)
+                inv = __fdividef(inv, 1.0f + __expf(-__bfloat162float(a.gate[(size_t)t * a.gate_stride + h])));
             const float* oc = a.ocos ? a.ocos + (size_t)a.tok_pos[t] * (DV / 2) + tid4 : nullptr;
             const float* os = a.ocos ? a.osin + (size_t)a.tok_pos[t] * (DV / 2) + tid4 : nullptr;
-            __nv_bfloat16* dst = a.out + ((size_t)t * a.nh + h) * DV + tid4 * 2;
-            const __nv_bfloat16* gt = a.gate ? a.gate + (size_t)t * a.gate_stride + (size_t)h * DV + tid4 * 2 : nullptr;
+            __nv_bfloat16* dst = a.out + (size_t)t * a.ldo + (size_t)h * DV + tid4 * 2;
+            const __nv_bfloat16* gt = a.gate && !a.gate_per_head ? a.gate + (size_t)t * a.gate_stride + (size_t)h * DV + tid4 * 2 : nullptr;
 #pragma unroll
             for (int i = 0; i < DV / 8; ++i) {
                 float v0 = o[i][2 * r] * inv, v1 = o[i][2 * r + 1] * inv;
@@ -298,7 +303,8 @@ __global__ void attention_window_mma_merge_kernel(const float* __restrict__ part
                                                   const __nv_bfloat16* __restrict__ gate, int gate_stride, int nh, int dv,
                                                   int splits, const float* __restrict__ sinks,
                                                   const float* __restrict__ ocos, const float* __restrict__ osin,
-                                                  const int* __restrict__ tok_pos) {
+                                                  const int* __restrict__ tok_pos, int gate_per_head,
+                                                  float out_scale, int ldo) {
     pdl_sync();
     const int t = blockIdx.x, h = blockIdx.y;
     const float* p = partial + ((size_t)t * nh + h) * splits * (dv + 2);
@@ -326,8 +332,9 @@ __global__ void attention_window_mma_merge_kernel(const float* __restrict__ part
             const float co = ocos[(size_t)tok_pos[t] * (dv / 2) + (c >> 1)], si = osin[(size_t)tok_pos[t] * (dv / 2) + (c >> 1)];
             v = (c & 1) ? v * co - other * si : v * co + other * si;
         }
-        if (gate) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * gate_stride + (size_t)h * dv + c])));
-        out[((size_t)t * nh + h) * dv + c] = __float2bfloat16_rn(v);
+        if (gate)
+            v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * gate_stride + (gate_per_head ? (size_t)h : (size_t)h * dv + c)])));
+        out[(size_t)t * ldo + (size_t)h * dv + c] = __float2bfloat16_rn(v * out_scale);
     }
 }
 
@@ -347,8 +354,34 @@ static int window_mma_launch(const WinMmaArgs& a, int nt, cudaStream_t s) {
     if (rc || a.splits == 1) return rc;
     dim3 mgrid(nt, a.nh);
     TB_LAUNCH(attention_window_mma_merge_kernel, mgrid, DV < 128 ? 64 : 128, 0, s, a.partial, a.out, a.gate, a.gate_stride,
-              a.nh, DV, a.splits, a.sinks, a.ocos, a.osin, a.tok_pos);
+              a.nh, DV, a.splits, a.sinks, a.ocos, a.osin, a.tok_pos, a.gate_per_head, a.out_scale, a.ldo);
     return tb_last_error();
+}
+
+static int window_mma_entry(WinMmaArgs a, int nt, int dk, int dv, cudaStream_t s) {
+    if (a.nh <= 0 || a.nkvh <= 0 || a.nh % a.nkvh || a.tiles < 0 || a.window <= 0 || a.keep_first < 0 || a.splits < 1)
+        return TB_ERR_ARG;
+    if (a.chunk < 0 || (a.ocos && !a.osin)) return TB_ERR_ARG;
+    if (a.splits > 1 && !a.partial) return TB_ERR_ARG;
+    if (a.ldo == 0) a.ldo = a.nh * dv;
+    if (a.ldo < a.nh * dv) return TB_ERR_ARG;
+    if (a.nh / a.nkvh > WM_ROWS) return TB_ERR_UNSUPPORTED;
+    if (a.q_stride % 8 || a.ldo % 8 || (((uintptr_t)a.q | (uintptr_t)a.out | (uintptr_t)a.kc | (uintptr_t)a.vc) & 15))
+        return TB_ERR_UNSUPPORTED;
+    if (!a.gate_per_head && (a.gate_stride % 8 || ((uintptr_t)a.gate & 15))) return TB_ERR_UNSUPPORTED;
+    if (a.tiles == 0) return 0;
+#define WM_CASE(K, V) if (dk == K && dv == V) return window_mma_launch<K, V>(a, nt, s);
+    WM_CASE(32, 32)
+    WM_CASE(48, 48)
+    WM_CASE(64, 64)
+    WM_CASE(96, 96)
+    WM_CASE(128, 128)
+    WM_CASE(64, 128)
+    WM_CASE(128, 64)
+    WM_CASE(32, 96)
+    WM_CASE(128, 256)
+#undef WM_CASE
+    return TB_ERR_UNSUPPORTED;
 }
 
 extern "C" {
@@ -366,32 +399,31 @@ int tb_attention_window_mma_bf16(const void* q, void* out, const void* kc, const
                                  int gate_stride, int nh, int nkvh, int dk, int dv, int splits, int window,
                                  int keep_first, float scale, float softcap, int chunk, const float* sinks,
                                  const float* ocos, const float* osin, cudaStream_t s) {
-    if (nh <= 0 || nkvh <= 0 || nh % nkvh || tiles < 0 || window <= 0 || keep_first < 0 || splits < 1) return TB_ERR_ARG;
-    if (chunk < 0 || (ocos && !osin)) return TB_ERR_ARG;
-    if (splits > 1 && !partial) return TB_ERR_ARG;
-    if (nh / nkvh > WM_ROWS) return TB_ERR_UNSUPPORTED;
-    if (q_stride % 8 || gate_stride % 8 ||
-        (((uintptr_t)q | (uintptr_t)out | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)gate) & 15))
-        return TB_ERR_UNSUPPORTED;
-    if (tiles == 0) return 0;
-    WinMmaArgs a{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
-                 (const __nv_bfloat16*)gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, ocos, osin,
-                 chunk, tiles, max_pages,
-                 q_stride, gate_stride, nh, nkvh, splits, window, keep_first, scale, softcap};
-#define WM_CASE(K, V) if (dk == K && dv == V) return window_mma_launch<K, V>(a, nt, s);
-    WM_CASE(32, 32)
-    WM_CASE(48, 48)
-    WM_CASE(64, 64)
-    WM_CASE(96, 96)
-    WM_CASE(128, 128)
-    WM_CASE(64, 128)
-    WM_CASE(128, 64)
-    WM_CASE(32, 96)
-    WM_CASE(128, 256)
-#undef WM_CASE
-    return TB_ERR_UNSUPPORTED;
+    return window_mma_entry(
+        WinMmaArgs{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
+                   (const __nv_bfloat16*)gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, ocos,
+                   osin, chunk, tiles, max_pages, q_stride, gate_stride, nh, nkvh, splits, window, keep_first, scale,
+                   softcap},
+        nt, dk, dv, s);
+}
+// The same with a gate of one number per (token, head) (gate_per_head), a multiplier of the output and a row pitch of
+// the output, for a mixer whose result lands in a wider row.
+int tb_attention_window_mma_heads_bf16(const void* q, void* out, const void* kc, const void* vc, const void* gate,
+                                 const int* tile_seq, const int* tile_t0, const int* tile_nq, const int* tok_pos,
+                                 const int* page_table, float* partial, int tiles, int nt, int max_pages, int q_stride,
+                                 int gate_stride, int nh, int nkvh, int dk, int dv, int splits, int window,
+                                 int keep_first, float scale, float softcap, int chunk, const float* sinks,
+                                 const float* ocos, const float* osin, int gate_per_head,
+                                 float out_scale, int ldo, cudaStream_t s) {
+    return window_mma_entry(
+        WinMmaArgs{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
+                   (const __nv_bfloat16*)gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, ocos,
+                   osin, chunk, tiles, max_pages, q_stride, gate_stride, nh, nkvh, splits, window, keep_first, scale,
+                   softcap, gate_per_head, out_scale, ldo},
+        nt, dk, dv, s);
 }
 }
 
 #include "tape.h"
 TB_TAPE_REGISTER(tb_attention_window_mma_bf16)
+TB_TAPE_REGISTER(tb_attention_window_mma_heads_bf16)

@@ -122,15 +122,19 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
 
 // ---- gated activations of a feed-forward's (gate, up) pair ------------------------------------------
 // kind 0: silu(g) * u.   kind 1: g' = min(g, limit), u' = clamp(u, -limit, limit);  g' * sigmoid(alpha g') * (u' + 1).
+// kind 3: gelu(g) * u with the tanh form of gelu, 0.5 g (1 + tanh(y)) = g / (1 + e^-2y), y = sqrt(2/pi) (g + 0.044715 g^3).
 // kind 2 stands beside them for a feed-forward WITHOUT a gate: a product of one matrix whose result passes
 // max(z, 0)^2 in the epilogue (TB_ACT_RELU2; the kernels apply it where they do not have a pair).
 #define TB_ACT_RELU2 2
+#define TB_GLU_GELU_TANH 3
 struct GluRule {
     int kind;
     float alpha, limit;
 };
+__device__ __forceinline__ float gelu_tanh_2y(float g) { return 1.5957691216057308f * (g + 0.044715f * g * g * g); }
 __device__ __forceinline__ float glu_apply(float g, float u, const GluRule r) {
     if (r.kind == 0) return g / (1.0f + expf(-g)) * u;
+    if (r.kind == TB_GLU_GELU_TANH) return g / (1.0f + expf(-gelu_tanh_2y(g))) * u;
     g = fminf(g, r.limit);
     u = fminf(fmaxf(u, -r.limit), r.limit);
     return g / (1.0f + expf(-r.alpha * g)) * (u + 1.0f);
@@ -138,6 +142,7 @@ __device__ __forceinline__ float glu_apply(float g, float u, const GluRule r) {
 // the same with the hardware's exponential and division (2 ulp), for results that are rounded to bfloat16 next
 __device__ __forceinline__ float glu_apply_fast(float g, float u, const GluRule r) {
     if (r.kind == 0) return __fdividef(g * u, 1.0f + __expf(-g));
+    if (r.kind == TB_GLU_GELU_TANH) return __fdividef(g * u, 1.0f + __expf(-gelu_tanh_2y(g)));
     g = fminf(g, r.limit);
     u = fminf(fmaxf(u, -r.limit), r.limit);
     return __fdividef(g * (u + 1.0f), 1.0f + __expf(-r.alpha * g));

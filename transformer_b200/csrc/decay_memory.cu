@@ -1,0 +1,558 @@
+// A linear memory with a decay per key channel made from the input, a bonus for the current token and a shift of the
+// input by one token (the time mixing of the RWKV family), state in float.
+//
+// Per head, with a state S [dim, dim] that is zero when a sequence starts (rows: key channels, columns: values):
+//
+//   o_t = S^T r_t + (r_t . (u k_t)) v_t;        S <- diag(w_t) S + k_t v_t^T;        w = exp(-exp(w0 + W2 tanh(a)))
+//
+// r, k, v, a and the output gate are projections of mixes of the token's input and the input of the token before:
+//   mix_m[t] = x[t] + (x[t - 1] - x[t]) mu_m        x[-1]: the sequence's last input of the step before (zeros at its start)
+//
+// State of one slot (floats): S [H][dim][dim], then the last input [width]; the pitch is a multiple of four.
+//
+//   shift_mix_kernel    all mixes of a token at once, and the group lists of the product that follows (a matrix per mix)
+//   decay_prep_kernel   prompts: decays and bonuses; one float record per (token, head) for the scan, r | k | w | bonus
+//   decay_scan_kernel   prompts: the recurrence token by token, a block = a sequence x a head x some columns of S, whose
+//                       rows are split over adjacent lanes, in registers; the lanes' sums meet only in the output, so
+//                       no token waits for another's reduction
+//   decay_step_kernel   one token per sequence: a block = a sequence x a head; decays, bonus, the state's way through the
+//                       registers, the head's norm and the gate in one kernel
+// Everything that enters the recurrence is float on both paths; x, r, k, v and the gate have the activations' type.
+#include "common.cuh"
+#include "attention_prefill.cuh"        // cp_async16, cp_async_commit, cp_async_wait
+
+constexpr int DM_MIXES = 5;             // r, k, v, gate, decay
+constexpr int DM_TOK = 4;               // tokens the scan stages per barrier
+constexpr int DM_SCAN = 128;            // threads of a scan block
+constexpr int DM_PREP_TOK = 8;          // tokens of a prep block
+
+__host__ __device__ inline int dm_rows(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+__host__ __device__ inline int dm_record(int dim) { return 3 * dm_rows(dim) + 4; }
+__host__ __device__ inline int dm_vpitch(int dim) { return (dim + 31) / 32 * 32; }
+__host__ __device__ inline long long dm_state(int H, int dim, int width) { return ((long long)H * dim * dim + width + 3) / 4 * 4; }
+
+// ---- the mixes ---------------------------------------------------------------------------------------------
+template <typename T, bool VEC, int TILE>
+__global__ void __launch_bounds__(128)
+shift_mix_kernel(const T* __restrict__ x, const float* __restrict__ mu, const float* __restrict__ state,
+                 long long pitch, long long at, T* __restrict__ out, int* __restrict__ offsets,
+                 int* __restrict__ row_group, int groups, const int* __restrict__ tok_seq,
+                 const int* __restrict__ seq_start, const int* __restrict__ slots, int nt, int d) {
+    constexpr int V = VEC ? 8 : 1;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    float m[DM_MIXES][V];
+#pragma unroll
+    for (int j = 0; j < DM_MIXES; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) m[j][e] = 0.f;
+    if (c < d) {        // weights: nothing of the step writes them
+#pragma unroll
+        for (int j = 0; j < DM_MIXES; ++j) {
+            if constexpr (VEC) load8(mu + (size_t)j * d + c, m[j]);
+            else m[j][0] = mu[(size_t)j * d + c];
+        }
+    }
+    pdl_sync();
+    if (blockIdx.x == 0 && blockIdx.y == 0) {
+        for (int j = threadIdx.x; j <= groups; j += blockDim.x) offsets[j] = j * nt;
+        if (row_group)
+            for (int j = threadIdx.x; j < groups * nt; j += blockDim.x) row_group[j] = j / nt;
+    }
+    if (c >= d) return;
+    const int t0 = blockIdx.x * TILE;
+    float before[V], now[V];
+#pragma unroll
+    for (int tt = 0; tt < TILE; ++tt) {
+        const int t = t0 + tt;
+        if (t >= nt) break;
+        const int b = tok_seq[t];
+        if constexpr (VEC) load8(x + (size_t)t * d + c, now);
+        else now[0] = ldf(x + (size_t)t * d + c);
+        if (t == seq_start[b]) {
+            const float* last = state + (size_t)slots[b] * pitch + at + c;
+#pragma unroll
+            for (int e = 0; e < V; ++e) before[e] = last[e];
+        } else if (tt == 0) {
+            if constexpr (VEC) load8(x + (size_t)(t - 1) * d + c, before);
+            else before[0] = ldf(x + (size_t)(t - 1) * d + c);
+        }
+#pragma unroll
+        for (int j = 0; j < DM_MIXES; ++j) {
+            float y[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) y[e] = now[e] + (before[e] - now[e]) * m[j][e];
+            T* dst = out + ((size_t)j * nt + t) * d + c;
+            if constexpr (VEC) store8(dst, y);
+            else stf(dst, y[0]);
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) before[e] = now[e];
+    }
+}
+
+template <typename T>
+static int shift_mix_launch(const void* x, const float* mu, const float* state, long long pitch, long long at, void* out,
+                            int* offsets, int* row_group, int groups, const int* tok_seq, const int* seq_start,
+                            const int* slots, int nt, int d, cudaStream_t s) {
+    if (nt < 0 || d <= 0 || groups < 1 || !offsets) return TB_ERR_ARG;
+    if (nt == 0) return 0;
+    const bool vec = d % 8 == 0 && (((uintptr_t)x | (uintptr_t)mu | (uintptr_t)out) & 15) == 0;
+    const int per = 128 * (vec ? 8 : 1), cols = (d + per - 1) / per;
+    const bool tiled = nt >= 256;
+    const dim3 grid(tiled ? (nt + 3) / 4 : nt, cols);
+#define SHIFT_GO(VEC, TILE)                                                                                           \
+    TB_LAUNCH((shift_mix_kernel<T, VEC, TILE>), grid, 128, 0, s, (const T*)x, mu, state, pitch, at, (T*)out, offsets, \
+              row_group, groups, tok_seq, seq_start, slots, nt, d)
+    if (vec && tiled) SHIFT_GO(true, 4);
+    else if (vec) SHIFT_GO(true, 1);
+    else if (tiled) SHIFT_GO(false, 4);
+    else SHIFT_GO(false, 1);
+#undef SHIFT_GO
+    return tb_last_error();
+}
+
+// ---- decays ------------------------------------------------------------------------------------------------
+// w0 + W2 row . ta for DT tokens at once; ta [DT][rank] in shared memory
+template <typename T, int DT>
+__device__ __forceinline__ void decay_dot(const T* __restrict__ w2row, const float* ta, int rank, float base,
+                                          float (&acc)[DT]) {
+#pragma unroll
+    for (int p = 0; p < DT; ++p) acc[p] = base;
+    if ((rank & 7) == 0) {
+        for (int q = 0; q < rank; q += 8) {
+            float w[8];
+            load8(w2row + q, w);
+#pragma unroll
+            for (int p = 0; p < DT; ++p) {
+                const float4 t0 = *reinterpret_cast<const float4*>(ta + p * rank + q);
+                const float4 t1 = *reinterpret_cast<const float4*>(ta + p * rank + q + 4);
+                acc[p] += w[0] * t0.x + w[1] * t0.y + w[2] * t0.z + w[3] * t0.w + w[4] * t1.x + w[5] * t1.y + w[6] * t1.z +
+                          w[7] * t1.w;
+            }
+        }
+        return;
+    }
+    for (int q = 0; q < rank; ++q) {
+        const float w = ldf(w2row + q);
+#pragma unroll
+        for (int p = 0; p < DT; ++p) acc[p] += w * ta[p * rank + q];
+    }
+}
+
+struct DecayArgs {
+    const void* z;          // [4 nt, H dim]: r, k, v, gate, nt rows each
+    const float* a;         // [nt, lda] the decay's first projection
+    const void* w2;         // [H dim, rank]
+    const float* w0;        // [H dim]
+    const float* u;         // [H dim]
+    float* rec;             // [nt, H, dm_record]
+    float* vals;            // [nt, H, dm_vpitch]
+    int nt, lda, H, dim, rank;
+};
+
+// A block = DM_PREP_TOK consecutive tokens x one head; a thread takes a key channel (or every 256th).
+template <typename T>
+__global__ void __launch_bounds__(256) decay_prep_kernel(const DecayArgs p) {
+    pdl_sync();
+    extern __shared__ __align__(16) float dm_sm[];        // [DM_PREP_TOK][rank] tanh(a)
+    __shared__ float part[8][DM_PREP_TOK];
+    const int t0 = blockIdx.x * DM_PREP_TOK, h = blockIdx.y;
+    const int n = min(DM_PREP_TOK, p.nt - t0), dim = p.dim, hd = p.H * dim;
+    const int DP = dm_rows(dim), PER = dm_record(dim), VP = dm_vpitch(dim);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    for (int i = threadIdx.x; i < DM_PREP_TOK * p.rank; i += blockDim.x) {
+        const int tt = i / p.rank, q = i - tt * p.rank;
+        dm_sm[i] = tt < n ? tanhf(p.a[(size_t)(t0 + tt) * p.lda + q]) : 0.f;
+    }
+    __syncthreads();
+    const T* z = static_cast<const T*>(p.z);
+    float bonus[DM_PREP_TOK];
+#pragma unroll
+    for (int tt = 0; tt < DM_PREP_TOK; ++tt) bonus[tt] = 0.f;
+    for (int c = threadIdx.x; c < DP; c += blockDim.x) {
+        const bool live = c < dim;
+        const int hc = h * dim + c;
+        float acc[DM_PREP_TOK];
+        float uc = 0.f;
+        if (live) {
+            decay_dot<T, DM_PREP_TOK>(static_cast<const T*>(p.w2) + (size_t)hc * p.rank, dm_sm, p.rank, p.w0[hc], acc);
+            uc = p.u[hc];
+        }
+#pragma unroll
+        for (int tt = 0; tt < DM_PREP_TOK; ++tt) {
+            if (tt >= n) break;
+            const int t = t0 + tt;
+            float* r = p.rec + ((size_t)t * p.H + h) * PER;
+            float rv = 0.f, kv = 0.f, w = 1.f, vv = 0.f;
+            if (live) {
+                rv = ldf(z + (size_t)t * hd + hc);
+                kv = ldf(z + ((size_t)p.nt + t) * hd + hc);
+                vv = ldf(z + ((size_t)2 * p.nt + t) * hd + hc);
+                w = expf(-expf(acc[tt]));
+                bonus[tt] += rv * uc * kv;
+            }
+            r[c] = rv;
+            r[DP + c] = kv;
+            r[2 * DP + c] = w;
+            if (c < VP) p.vals[((size_t)t * p.H + h) * VP + c] = vv;
+        }
+    }
+    // VP may exceed DP only for dim <= 16
+    if (VP > DP)
+        for (int i = threadIdx.x; i < n * (VP - DP); i += blockDim.x)
+            p.vals[((size_t)(t0 + i / (VP - DP)) * p.H + h) * VP + DP + i % (VP - DP)] = 0.f;
+#pragma unroll
+    for (int tt = 0; tt < DM_PREP_TOK; ++tt) {
+        const float s = warp_sum(bonus[tt]);
+        if (lane == 0) part[warp][tt] = s;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < n * 4; i += blockDim.x) {
+        const int tt = i >> 2, j = i & 3;
+        float s = 0.f;
+        if (j == 0)
+            for (int w = 0; w < warps; ++w) s += part[w][tt];
+        p.rec[((size_t)(t0 + tt) * p.H + h) * PER + 3 * DP + j] = s;
+    }
+}
+
+// ---- the scan ------------------------------------------------------------------------------------------------
+struct DecayScanArgs {
+    const float* rec;
+    const float* vals;
+    float* state;           // [slots, pitch]
+    float* out;             // [nt, H dim]
+    const void* x;          // [nt, width]: a sequence's last row becomes its state's last input
+    const int* seq_start;
+    const int* slots;
+    long long pitch;
+    int H, dim, width;
+};
+
+// RPT rows of a column per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)), DM_SCAN / SPLIT columns a block.
+template <typename T, int RPT, int SPLIT>
+__global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs a) {
+    pdl_sync();
+    constexpr int DP = RPT * SPLIT;
+    constexpr int COLS = DM_SCAN / SPLIT;
+    constexpr int PER = 3 * DP + 4;
+    constexpr int ROW = PER + COLS;
+    constexpr int ROW4 = ROW / 4;
+    __shared__ __align__(16) float sm[2][DM_TOK][ROW];
+    const int b = blockIdx.x, h = blockIdx.y;
+    const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT;
+    const int col0 = blockIdx.z * COLS, col = col0 + cl;
+    const int dim = a.dim, H = a.H;
+    const bool has_col = col < dim;
+    const int t0 = a.seq_start[b], t1 = a.seq_start[b + 1];
+    if (t0 >= t1) return;
+    const int VP = dm_vpitch(dim);
+    float* slot = a.state + (size_t)a.slots[b] * a.pitch;
+    float* S = slot + (size_t)h * dim * dim;
+    float s[RPT];
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const int r = ((i >> 2) * SPLIT + part) * 4 + (i & 3);
+        s[i] = (r < dim && has_col) ? S[(size_t)r * dim + col] : 0.f;
+    }
+    auto issue = [&](int ts, int par) {
+        const int ntok = min(DM_TOK, t1 - ts);
+        for (int idx = tid; idx < ntok * ROW4; idx += DM_SCAN) {
+            const int tt = idx / ROW4, e4 = idx - tt * ROW4;
+            // columns behind the padded row of values are left alone: no column of the head reads them
+            if (e4 >= PER / 4 && col0 + (e4 - PER / 4) * 4 >= VP) continue;
+            const float* src = e4 < PER / 4 ? a.rec + ((size_t)(ts + tt) * H + h) * PER + e4 * 4
+                                            : a.vals + ((size_t)(ts + tt) * H + h) * VP + col0 + (e4 - PER / 4) * 4;
+            cp_async16((uint32_t)__cvta_generic_to_shared(&sm[par][tt][e4 * 4]), src);
+        }
+        cp_async_commit();
+    };
+    issue(t0, 0);
+    for (int ts = t0, st = 0; ts < t1; ts += DM_TOK, ++st) {
+        const int par = st & 1;
+        cp_async_wait<0>();
+        __syncthreads();            // this stage has landed for everyone, and everyone is done with the stage before
+        if (ts + DM_TOK < t1) issue(ts + DM_TOK, par ^ 1);
+        const int ntok = min(DM_TOK, t1 - ts);
+        float o[DM_TOK];
+#pragma unroll
+        for (int tt = 0; tt < DM_TOK; ++tt) {
+            o[tt] = 0.f;
+            if (tt >= ntok) continue;
+            const float* row = &sm[par][tt][0];
+            const float4* R4 = reinterpret_cast<const float4*>(row);
+            const float4* K4 = reinterpret_cast<const float4*>(row + DP);
+            const float4* W4 = reinterpret_cast<const float4*>(row + 2 * DP);
+            const float v = row[PER + cl];
+            float d4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int i4 = 0; i4 < RPT / 4; ++i4) {
+                const int ch = i4 * SPLIT + part;
+                const float4 r = R4[ch], k = K4[ch], w = W4[ch];
+                float* si = s + i4 * 4;
+                d4[0] += si[0] * r.x; d4[1] += si[1] * r.y; d4[2] += si[2] * r.z; d4[3] += si[3] * r.w;
+                si[0] = si[0] * w.x + k.x * v; si[1] = si[1] * w.y + k.y * v;
+                si[2] = si[2] * w.z + k.z * v; si[3] = si[3] * w.w + k.w * v;
+            }
+            o[tt] = (d4[0] + d4[1]) + (d4[2] + d4[3]);
+        }
+#pragma unroll
+        for (int tt = 0; tt < DM_TOK; ++tt)
+#pragma unroll
+            for (int q = 1; q < SPLIT; q <<= 1) o[tt] += __shfl_xor_sync(0xffffffffu, o[tt], q);
+#pragma unroll
+        for (int tt = 0; tt < DM_TOK; ++tt)
+            if (tt < ntok && part == (tt & (SPLIT - 1)) && has_col) {
+                const float* row = &sm[par][tt][0];
+                a.out[((size_t)(ts + tt) * H + h) * dim + col] = o[tt] + row[3 * DP] * row[PER + cl];
+            }
+    }
+#pragma unroll
+    for (int i = 0; i < RPT; ++i) {
+        const int r = ((i >> 2) * SPLIT + part) * 4 + (i & 3);
+        if (r < dim && has_col) S[(size_t)r * dim + col] = s[i];
+    }
+    if (h == 0 && blockIdx.z == 0) {        // the mixes have read the old one
+        const T* last = static_cast<const T*>(a.x) + (size_t)(t1 - 1) * a.width;
+        float* to = slot + (size_t)H * dim * dim;
+        for (int c = tid; c < a.width; c += DM_SCAN) to[c] = ldf(last + c);
+    }
+}
+
+static int dm_lanes_override = 0;       // measurements: lanes per column whatever the batch (0: by the rule below)
+
+template <typename T, int RPT, int SPLIT>
+static void decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
+    dim3 grid(B, a.H, (a.dim + DM_SCAN / SPLIT - 1) / (DM_SCAN / SPLIT));
+    if (early)
+        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT>), grid, DM_SCAN, 0, s, a);
+    else        // prompts: the blocks run for the whole sequence and want an SM each (see tb_launch_plain)
+        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT>, grid, dim3(DM_SCAN), 0, s, a);
+}
+
+template <typename T>
+static int decay_scan_launch(const DecayScanArgs& a, int nt, int B, cudaStream_t s) {
+    if (B < 0 || a.H <= 0 || a.dim <= 0 || a.width <= 0 || a.pitch < dm_state(a.H, a.dim, a.width)) return TB_ERR_ARG;
+    if (a.dim > 256) return TB_ERR_UNSUPPORTED;
+    if (B == 0) return 0;
+    const int rows = dm_rows(a.dim);
+    int lanes = rows >= 128 ? 16 : rows >= 32 ? 8 : 4;
+    if (dm_lanes_override > 0) lanes = dm_lanes_override;
+    const bool early = nt <= 2 * B;
+    if (lanes > rows / 4) lanes = rows / 4;
+    if (rows / lanes > 32) lanes = rows / 32;
+    switch (rows / lanes * 100 + lanes) {       // rows per thread, lanes per column
+        case 4 * 100 + 4: decay_scan_go<T, 4, 4>(a, B, early, s); break;
+        case 8 * 100 + 4: decay_scan_go<T, 8, 4>(a, B, early, s); break;
+        case 4 * 100 + 8: decay_scan_go<T, 4, 8>(a, B, early, s); break;
+        case 16 * 100 + 4: decay_scan_go<T, 16, 4>(a, B, early, s); break;
+        case 8 * 100 + 8: decay_scan_go<T, 8, 8>(a, B, early, s); break;
+        case 4 * 100 + 16: decay_scan_go<T, 4, 16>(a, B, early, s); break;
+        case 32 * 100 + 4: decay_scan_go<T, 32, 4>(a, B, early, s); break;
+        case 16 * 100 + 8: decay_scan_go<T, 16, 8>(a, B, early, s); break;
+        case 8 * 100 + 16: decay_scan_go<T, 8, 16>(a, B, early, s); break;
+        case 32 * 100 + 8: decay_scan_go<T, 32, 8>(a, B, early, s); break;
+        case 16 * 100 + 16: decay_scan_go<T, 16, 16>(a, B, early, s); break;
+        default: return TB_ERR_UNSUPPORTED;
+    }
+    return tb_last_error();
+}
+
+template <typename T>
+static int decay_prep_launch(const DecayArgs& p, cudaStream_t s) {
+    if (p.nt < 0 || p.H <= 0 || p.dim <= 0 || p.rank <= 0 || p.lda < p.rank) return TB_ERR_ARG;
+    if (p.dim > 256) return TB_ERR_UNSUPPORTED;
+    const size_t smem = (size_t)DM_PREP_TOK * p.rank * sizeof(float);
+    if (smem > 48 * 1024 || (p.rank % 8 == 0 && ((uintptr_t)p.w2 & 15))) return TB_ERR_UNSUPPORTED;
+    if (p.nt == 0) return 0;
+    TB_LAUNCH((decay_prep_kernel<T>), dim3((p.nt + DM_PREP_TOK - 1) / DM_PREP_TOK, p.H), max(32, dm_rows(p.dim)), smem, s, p);
+    return tb_last_error();
+}
+
+// ---- one token per sequence -------------------------------------------------------------------------------------
+struct DecayStepArgs {
+    const void* z;          // [4 nt, H dim]: r, k, v, gate, nt rows each
+    const void* x;          // [nt, width]
+    const float* a;         // [nt, lda]
+    const void* w2;
+    const float* w0;
+    const float* u;
+    const float* norm;      // [H dim]
+    float* state;
+    void* y;                // [nt, ldy]
+    const int* seq_start;
+    const int* slots;
+    long long pitch;
+    int nt, width, lda, ldy, H, dim, rank;
+    float eps;
+};
+
+// VEC: four columns a thread and access (dim a multiple of four), else one.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) {
+    constexpr int V = VEC ? 4 : 1;
+    constexpr int U = VEC ? 4 : 8;          // rows asked for together
+    extern __shared__ __align__(16) float dm_sm[];
+    const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    const int dim = p.dim, hd = p.H * dim, rank4 = (p.rank + 3) / 4 * 4, dim4 = (dim + 3) / 4 * 4;
+    const int nc = dim / V, G = 256 / nc;   // columns' threads, groups of rows
+    float* ta = dm_sm;                      // [rank4]
+    float* r_s = ta + rank4;                // [dim4] each
+    float* k_s = r_s + dim4;
+    float* w_s = k_s + dim4;
+    float* v_s = w_s + dim4;
+    float* o_s = v_s + dim4;                // [G][dim4]
+    __shared__ float red[33];
+    const int hc = h * dim + tid;
+    float w0 = 0.f, u = 0.f, nw = 0.f;
+    if (tid < dim) {                        // weights: nothing of the step writes them
+        w0 = p.w0[hc];
+        u = p.u[hc];
+        nw = p.norm[hc];
+    }
+    pdl_sync();
+    const int t = p.seq_start[b];
+    float* slot = p.state + (size_t)p.slots[b] * p.pitch;
+    float* S = slot + (size_t)h * dim * dim;
+    const T* z = static_cast<const T*>(p.z);
+    for (int q = tid; q < p.rank; q += 256) ta[q] = tanhf(p.a[(size_t)t * p.lda + q]);
+    float bonus = 0.f, gate = 0.f;
+    if (tid < dim) {
+        const float r = ldf(z + (size_t)t * hd + hc), k = ldf(z + ((size_t)p.nt + t) * hd + hc);
+        r_s[tid] = r;
+        k_s[tid] = k;
+        v_s[tid] = ldf(z + ((size_t)2 * p.nt + t) * hd + hc);
+        gate = ldf(z + ((size_t)3 * p.nt + t) * hd + hc);
+        bonus = r * u * k;
+    }
+    __syncthreads();
+    if (tid < dim) {
+        float acc[1];
+        decay_dot<T, 1>(static_cast<const T*>(p.w2) + (size_t)hc * p.rank, ta, p.rank, w0, acc);
+        w_s[tid] = expf(-expf(acc[0]));
+    }
+    bonus = block_sum(bonus, red);          // (and everyone's part of w_s is there)
+    const int rg = tid / nc, c = (tid - rg * nc) * V;
+    if (rg < G) {
+        float acc[V], v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            acc[e] = 0.f;
+            v[e] = v_s[c + e];
+        }
+        for (int r0 = rg; r0 < dim; r0 += G * U) {
+            float s[U][V];
+#pragma unroll
+            for (int q = 0; q < U; ++q) {
+                const int r = r0 + q * G;
+                if (r < dim) {
+                    if constexpr (VEC) {
+                        const float4 f = *reinterpret_cast<const float4*>(S + (size_t)r * dim + c);
+                        s[q][0] = f.x; s[q][1] = f.y; s[q][2] = f.z; s[q][3] = f.w;
+                    } else {
+                        s[q][0] = S[(size_t)r * dim + c];
+                    }
+                }
+            }
+#pragma unroll
+            for (int q = 0; q < U; ++q) {
+                const int r = r0 + q * G;
+                if (r >= dim) break;
+                const float rr = r_s[r], kk = k_s[r], ww = w_s[r];
+#pragma unroll
+                for (int e = 0; e < V; ++e) {
+                    acc[e] += s[q][e] * rr;
+                    s[q][e] = s[q][e] * ww + kk * v[e];
+                }
+                if constexpr (VEC)
+                    *reinterpret_cast<float4*>(S + (size_t)r * dim + c) = make_float4(s[q][0], s[q][1], s[q][2], s[q][3]);
+                else
+                    S[(size_t)r * dim + c] = s[q][0];
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) o_s[rg * dim4 + c + e] = acc[e];
+    }
+    __syncthreads();
+    float o = 0.f;
+    if (tid < dim) {
+        for (int g = 0; g < G; ++g) o += o_s[g * dim4 + tid];
+        o += bonus * v_s[tid];
+    }
+    const float rs = 1.0f / sqrtf(block_sum(o * o, red) / (float)dim + p.eps);
+    if (tid < dim) stf(static_cast<T*>(p.y) + (size_t)t * p.ldy + hc, o * rs * nw * (gate / (1.0f + expf(-gate))));
+    if (h == 0) {                           // the mixes have read the old one
+        const T* row = static_cast<const T*>(p.x) + (size_t)t * p.width;
+        float* to = slot + (size_t)p.H * dim * dim;
+        for (int q = tid; q < p.width; q += 256) to[q] = ldf(row + q);
+    }
+}
+
+template <typename T>
+static int decay_step_launch(const DecayStepArgs& p, int B, cudaStream_t s) {
+    if (B < 0 || p.nt < B || p.H <= 0 || p.dim <= 0 || p.rank <= 0 || p.lda < p.rank || p.ldy < p.H * p.dim ||
+        p.pitch < dm_state(p.H, p.dim, p.width))
+        return TB_ERR_ARG;
+    if (p.dim > 256 || p.rank > 4096 || (p.rank % 8 == 0 && ((uintptr_t)p.w2 & 15))) return TB_ERR_UNSUPPORTED;
+    if (B == 0) return 0;
+    const bool vec = p.dim % 4 == 0 && p.pitch % 4 == 0 && ((uintptr_t)p.state & 15) == 0;
+    const int dim4 = (p.dim + 3) / 4 * 4, G = 256 / (p.dim / (vec ? 4 : 1));
+    const size_t smem = ((size_t)(p.rank + 3) / 4 * 4 + (size_t)(4 + G) * dim4) * sizeof(float);
+    if (smem > 48 * 1024) return TB_ERR_UNSUPPORTED;
+    if (vec) TB_LAUNCH((decay_step_kernel<T, true>), dim3(B, p.H), 256, smem, s, p);
+    else TB_LAUNCH((decay_step_kernel<T, false>), dim3(B, p.H), 256, smem, s, p);
+    return tb_last_error();
+}
+
+extern "C" {
+// Floats of state per slot.
+int tb_decay_state_size(int H, int dim, int width) { return (int)dm_state(H, dim, width); }
+int tb_decay_record_size(int dim) { return dm_record(dim); }
+int tb_decay_value_pitch(int dim) { return dm_vpitch(dim); }
+// For measurements: lanes per column in the scan whatever the batch; 0 gives the choice back to the rule.
+int tb_decay_scan_lanes(int lanes) {
+    dm_lanes_override = lanes;
+    return 0;
+}
+// out [5, nt, d]: the mixes of every token; offsets [groups + 1] and row_group [groups nt] (may be null): the lists by
+// which one grouped product multiplies the first `groups` of them with a matrix each.  `at`: where in a slot's state the
+// last input lies.
+#define TB_DECAY(SFX, T)                                                                                              \
+    int tb_shift_mix_##SFX(const void* x, const float* mu, const float* state, long long pitch, long long at,         \
+                           void* out, int* offsets, int* row_group, int groups, const int* tok_seq,                   \
+                           const int* seq_start, const int* slots, int nt, int d, cudaStream_t s) {                   \
+        return shift_mix_launch<T>(x, mu, state, pitch, at, out, offsets, row_group, groups, tok_seq, seq_start,      \
+                                   slots, nt, d, s);                                                                  \
+    }                                                                                                                 \
+    int tb_decay_prep_##SFX(const void* z, const float* a, int lda, const void* w2, const float* w0, const float* u,  \
+                            float* rec, float* vals, int nt, int H, int dim, int rank, cudaStream_t s) {              \
+        if (((uintptr_t)rec | (uintptr_t)vals) & 15) return TB_ERR_ARG;                                               \
+        return decay_prep_launch<T>(DecayArgs{z, a, w2, w0, u, rec, vals, nt, lda, H, dim, rank}, s);                 \
+    }                                                                                                                 \
+    int tb_decay_scan_##SFX(const float* rec, const float* vals, float* state, long long pitch, float* out,           \
+                            const void* x, int width, const int* seq_start, const int* slots, int nt, int B, int H,   \
+                            int dim, cudaStream_t s) {                                                                \
+        if (((uintptr_t)rec | (uintptr_t)vals) & 15) return TB_ERR_ARG;                                               \
+        return decay_scan_launch<T>(DecayScanArgs{rec, vals, state, out, x, seq_start, slots, pitch, H, dim, width},  \
+                                    nt, B, s);                                                                        \
+    }                                                                                                                 \
+    int tb_decay_step_##SFX(const void* z, const void* x, int width, const float* a, int lda, const void* w2,         \
+                            const float* w0, const float* u, const float* norm, float eps, float* state,              \
+                            long long pitch, void* y, int ldy, const int* seq_start, const int* slots, int nt, int B, \
+                            int H, int dim, int rank, cudaStream_t s) {                                               \
+        return decay_step_launch<T>(DecayStepArgs{z, x, a, w2, w0, u, norm, state, y, seq_start, slots, pitch, nt,    \
+                                                  width, lda, ldy, H, dim, rank, eps}, B, s);                         \
+    }
+TB_DECAY(f32, float)
+TB_DECAY(bf16, __nv_bfloat16)
+}
+
+#include "tape.h"
+TB_TAPE_REGISTER(tb_shift_mix_f32)
+TB_TAPE_REGISTER(tb_shift_mix_bf16)
+TB_TAPE_REGISTER(tb_decay_prep_f32)
+TB_TAPE_REGISTER(tb_decay_prep_bf16)
+TB_TAPE_REGISTER(tb_decay_scan_f32)
+TB_TAPE_REGISTER(tb_decay_scan_bf16)
+TB_TAPE_REGISTER(tb_decay_step_f32)
+TB_TAPE_REGISTER(tb_decay_step_bf16)

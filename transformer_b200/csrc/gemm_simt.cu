@@ -216,14 +216,15 @@ extern "C" {
 TB_GEMM(tb_gemm_simt_f32, float)
 TB_GEMM(tb_gemm_simt_bf16, __nv_bfloat16)
 
-// The (gate, up) pair product with the clamped form of the gate: g' = min(g, limit), u' = clamp(u, -limit, limit),
-// C = g' * sigmoid(alpha g') * (u' + 1).
+// The (gate, up) pair product with another form of the pair than silu(g) u (see GluRule): kind 1 the clamped form with
+// alpha and limit, kind 3 the tanh form of gelu on the gate.
 #define TB_GEMM_GLU(NAME, T)                                                                                    \
     int NAME(const void* A, const int* a_rows, const void* B, void* C, const int* group_offsets,               \
              long long b_group_stride, int lda, int ldb, int ldc, int M, int N, int K, int G, float alpha,     \
-             float limit, cudaStream_t s) {                                                                     \
+             float limit, int kind, cudaStream_t s) {                                                           \
+        if (kind != 1 && kind != TB_GLU_GELU_TANH) return TB_ERR_ARG;                                           \
         GemmArgs a{A, a_rows, B, C, group_offsets, b_group_stride, lda, ldb, ldc, M, N, K, G,                   \
-                   GluRule{1, alpha, limit}, 0, 0};                                                             \
+                   GluRule{kind, alpha, limit}, 0, 0};                                                             \
         return gemm_simt_launch<T, T, true>(a, s);                                                              \
     }
 TB_GEMM_GLU(tb_gemm_simt_glu_f32, float)

@@ -327,13 +327,14 @@ int tb_gemm_skinny_bf16(const void* X, const int* x_rows, const void* W, void* Y
                         max_group_rows, row_group, x_div, w_constant,
                         GluRule{out_kind == 3 ? TB_ACT_RELU2 : 0, 0.f, 0.f}, s);
 }
-// The (gate, up) pair product with the clamped form of the gate (see GluRule, kind 1).
+// The (gate, up) pair product with another form of the pair (see GluRule, kinds 1 and 3).
 int tb_gemm_skinny_glu_bf16(const void* X, const int* x_rows, const void* W, void* Y, const int* group_offsets,
                             long long w_group_stride, int ldx, int ldw, int ldy, int M, int N, int K, int G,
                             int max_group_rows, const int* row_group, int x_div, int w_constant, float alpha,
-                            float limit, cudaStream_t s) {
+                            float limit, int kind, cudaStream_t s) {
+    if (kind != 1 && kind != TB_GLU_GELU_TANH) return TB_ERR_ARG;
     return skinny_entry(X, x_rows, W, Y, group_offsets, w_group_stride, ldx, ldw, ldy, M, N, K, G, 2, max_group_rows,
-                        row_group, x_div, w_constant, GluRule{1, alpha, limit}, s);
+                        row_group, x_div, w_constant, GluRule{kind, alpha, limit}, s);
 }
 }
 

@@ -559,10 +559,11 @@ int tb_gemm_tc_bf16(const void* A, const void* B, void* C, const int* group_offs
                     int N, int K, int G, int out_kind, cudaStream_t s) {
     return gemm_tc_entry(A, B, C, group_offsets, lda, ldb, ldc, M, N, K, G, out_kind, GluRule{0, 0.f, 0.f}, s);
 }
-// The (gate, up) pair product with the clamped form of the gate (see GluRule, kind 1).
+// The (gate, up) pair product with another form of the pair (see GluRule, kinds 1 and 3).
 int tb_gemm_tc_glu_bf16(const void* A, const void* B, void* C, const int* group_offsets, int lda, int ldb, int ldc,
-                        int M, int N, int K, int G, float alpha, float limit, cudaStream_t s) {
-    return gemm_tc_entry(A, B, C, group_offsets, lda, ldb, ldc, M, N, K, G, 2, GluRule{1, alpha, limit}, s);
+                        int M, int N, int K, int G, float alpha, float limit, int kind, cudaStream_t s) {
+    if (kind != 1 && kind != TB_GLU_GELU_TANH) return TB_ERR_ARG;
+    return gemm_tc_entry(A, B, C, group_offsets, lda, ldb, ldc, M, N, K, G, 2, GluRule{kind, alpha, limit}, s);
 }
 
 // Nonzero if any tensor-core product gave up on a wait since the last call (1 producer, 2 MMA,

@@ -11,6 +11,9 @@
 //   queries go to `qout`, keys and values into the paged cache
 //
 // The convolution, the norm, the temperature and the rotations are optional (taps = 1, null weights, null tables).
+// A second launcher (tb_head_prep_keyed) runs the same kernels for heads whose values are their keys:
+//   u = z + bias,   q_h <- u_q,h / rms(u_q,h),  k_g <- u_k,g / rms(u_k,g)  without weights,   v_g = u_k,g as it is
+// A rotation leaves a head's root mean square as it was, so the norm may stand on either side of it.
 // Everything is float; one rounding at each store.
 //
 // A warp takes ONE head (a query, key or value head) of a tile of consecutive tokens; a lane holds the pairs
@@ -52,6 +55,9 @@ struct HeadPrepArgs {
     float eps;
     float* vfirst;          // [nt, nkvh * dv] or null: the values of the blend's source
     const float* vmix;      // one number, or null
+    const float* bias = nullptr;    // [(nh + nkvh) dk], added to the projections, or null
+    int values_are_keys = 0;        // value head g reads key head g's columns
+    int unit = 0;                   // queries and keys are normed without weights
 };
 
 // two neighbouring entries, as one access where the layout allows it
@@ -93,7 +99,9 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
     const int C = (a.nh + a.nkvh) * a.dk + a.nkvh * a.dv;
     const int kind = h < a.nh ? 0 : h < a.nh + a.nkvh ? 1 : 2;             // query, key, value
     const int dim = kind == 2 ? a.dv : a.dk;
-    const int coff = kind == 2 ? (a.nh + a.nkvh) * a.dk + (h - a.nh - a.nkvh) * a.dv : h * a.dk;
+    const int coff = kind < 2 ? h * a.dk : a.values_are_keys ? (h - a.nkvh) * a.dk
+                                         : (a.nh + a.nkvh) * a.dk + (h - a.nh - a.nkvh) * a.dv;
+    const bool normed = kind < 2 && (a.unit || (kind == 0 ? a.wq : a.wk));
     if ((kind == 1 && !a.kc) || (kind == 2 && !a.vc)) {
         if (!(a.decode && a.conv && a.taps > 1)) return;                   // nothing to write, no state to move on
     }
@@ -128,6 +136,10 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
             const int c = coff + 2 * i;
             float o0, o1;
             ld2<T, VEC>(z + (size_t)t * a.ldz + c, two, o0, o1);
+            if (a.bias) {
+                o0 += a.bias[c];
+                if (two) o1 += a.bias[c + 1];
+            }
             float a0 = o0, a1 = o1;
             if (conv) {
                 a0 = a1 = 0.f;
@@ -196,7 +208,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32) head_prep_kernel(const HeadPrep
             dst = base + (((size_t)page * a.nkvh + g) * TB_PAGE + pos % TB_PAGE) * dim;
         }
         float rs = 1.f;
-        if (w) rs = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+        if (normed) rs = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
         if (kind == 0 && a.temp) rs *= a.temp[h];
 #pragma unroll
         for (int r = 0; r < HP_PAIRS; ++r) {
@@ -233,7 +245,9 @@ __global__ void __launch_bounds__(HP_WARPS * 32, PAIRS <= 2 ? 6 : 3) head_prep_t
     const int C = (a.nh + a.nkvh) * a.dk + a.nkvh * a.dv;
     const int kind = h < a.nh ? 0 : h < a.nh + a.nkvh ? 1 : 2;             // query, key, value
     const int dim = kind == 2 ? a.dv : a.dk;
-    const int coff = kind == 2 ? (a.nh + a.nkvh) * a.dk + (h - a.nh - a.nkvh) * a.dv : h * a.dk;
+    const int coff = kind < 2 ? h * a.dk : a.values_are_keys ? (h - a.nkvh) * a.dk
+                                         : (a.nh + a.nkvh) * a.dk + (h - a.nh - a.nkvh) * a.dv;
+    const bool normed = kind < 2 && (a.unit || (kind == 0 ? a.wq : a.wk));
     if ((kind == 1 && !a.kc) || (kind == 2 && !a.vc)) return;
     constexpr int HIST = TAPS > 1 ? TAPS - 1 : 1;
     float wr[PAIRS][2 * TAPS];                      // wr[r][e * TAPS + j]: entry 2i + e of the head, tap j
@@ -259,11 +273,14 @@ __global__ void __launch_bounds__(HP_WARPS * 32, PAIRS <= 2 ? 6 : 3) head_prep_t
     const float* cosT = kind == 2 ? a.vcos : a.cosT;
     const float* sinT = kind == 2 ? a.vsin : a.sinT;
     float nw0[PAIRS], nw1[PAIRS];                     // the norm's weights of this lane's entries
+    float2 bias[PAIRS];
 #pragma unroll
     for (int r = 0; r < PAIRS; ++r) {
         const int i = lane + 32 * r;
         nw0[r] = (w && 2 * i < dim) ? w[2 * i] : 1.f;
         nw1[r] = (w && 2 * i < dim) ? w[2 * i + 1] : 1.f;
+        bias[r] = make_float2(0.f, 0.f);
+        if (a.bias && 2 * i < dim) bias[r] = make_float2(a.bias[coff + 2 * i], a.bias[coff + 2 * i + 1]);
     }
     const float temp_h = (kind == 0 && a.temp) ? a.temp[h] : 1.f;
     const int t0 = blockIdx.x * TILE;
@@ -339,7 +356,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32, PAIRS <= 2 ? 6 : 3) head_prep_t
         float ss = 0.f;
 #pragma unroll
         for (int r = 0; r < PAIRS; ++r) {
-            float a0 = wr[r][TAPS - 1] * own[tt][r].x, a1 = wr[r][2 * TAPS - 1] * own[tt][r].y;
+            float a0 = wr[r][TAPS - 1] * own[tt][r].x + bias[r].x, a1 = wr[r][2 * TAPS - 1] * own[tt][r].y + bias[r].y;
             if constexpr (TAPS > 1) {
 #pragma unroll
                 for (int j = 0; j < TAPS - 1; ++j) {
@@ -385,7 +402,7 @@ __global__ void __launch_bounds__(HP_WARPS * 32, PAIRS <= 2 ? 6 : 3) head_prep_t
             dst = static_cast<T*>(kind == 1 ? a.kc : a.vc) + (((size_t)page * a.nkvh + g) * TB_PAGE + pos % TB_PAGE) * dim;
         }
         float rs = 1.f;
-        if (w) rs = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+        if (normed) rs = 1.0f / sqrtf(warp_sum(ss) / (float)dim + a.eps);
         rs *= temp_h;
 #pragma unroll
         for (int r = 0; r < PAIRS; ++r) {
@@ -459,8 +476,44 @@ extern "C" {
     }
 TB_HEAD_PREP(f32, float)
 TB_HEAD_PREP(bf16, __nv_bfloat16)
+// Heads whose values are their keys: z holds q | k (and whatever follows), bias [(nh + nkvh) dk] or null; queries and
+// keys are normed per head without weights when `unit` says so.
+#define TB_HEAD_PREP_KEYED(SFX, T)                                                                                    \
+    int tb_head_prep_keyed_##SFX(const void* z, int ldz, const float* bias, int unit, float eps, const float* cosT,   \
+                                 const float* sinT, void* qout, void* kc, void* vc, const int* tok_seq,               \
+                                 const int* tok_pos, const int* seq_start, const int* page_table, int max_pages,      \
+                                 int nt, int nh, int nkvh, int dk, int rdims, cudaStream_t s) {                       \
+        if (nt < 0 || nh <= 0 || nkvh <= 0 || dk <= 0 || rdims < 0 || rdims > dk || rdims % 2) return TB_ERR_ARG;     \
+        if ((rdims && (!cosT || !sinT)) || ldz < (nh + nkvh) * dk) return TB_ERR_ARG;                                 \
+        if (dk > 64 * HP_PAIRS) return TB_ERR_UNSUPPORTED;                                                            \
+        if (nt == 0) return 0;                                                                                        \
+        const int groups = (nh + 2 * nkvh + HP_WARPS - 1) / HP_WARPS;                                                 \
+        const int tile = nt >= 64 ? 8 : 1;                                                                            \
+        HeadPrepArgs a{z, nullptr, nullptr, 0, nullptr, nullptr, nullptr, cosT, sinT, nullptr, nullptr, qout, kc, vc, \
+                       tok_seq, tok_pos, seq_start, nullptr, page_table, max_pages, ldz, nt, nh, nkvh, dk, dk, rdims, \
+                       1, 0, tile, 0, eps, nullptr, nullptr};                                                         \
+        a.bias = bias;                                                                                                \
+        a.values_are_keys = 1;                                                                                        \
+        a.unit = unit ? 1 : 0;                                                                                        \
+        const size_t es = sizeof(T);                                                                                  \
+        const bool vec = dk % 2 == 0 && ldz % 2 == 0 && (uintptr_t)z % (2 * es) == 0 &&                               \
+                         (uintptr_t)qout % (2 * es) == 0 && (uintptr_t)kc % (2 * es) == 0 &&                          \
+                         (uintptr_t)vc % (2 * es) == 0;                                                               \
+        if (vec && tile == 8) {                                                                                       \
+            head_prep_tile_launch<T, 1>(a, dim3((nt + HP_TILE - 1) / HP_TILE, groups), dk, s);                        \
+            return tb_last_error();                                                                                   \
+        }                                                                                                             \
+        const dim3 grid((nt + tile - 1) / tile, groups);                                                              \
+        if (vec) TB_LAUNCH((head_prep_kernel<T, true>), grid, HP_WARPS * 32, 0, s, a);                                \
+        else TB_LAUNCH((head_prep_kernel<T, false>), grid, HP_WARPS * 32, 0, s, a);                                   \
+        return tb_last_error();                                                                                       \
+    }
+TB_HEAD_PREP_KEYED(f32, float)
+TB_HEAD_PREP_KEYED(bf16, __nv_bfloat16)
 }
 
 #include "tape.h"
+TB_TAPE_REGISTER(tb_head_prep_keyed_f32)
+TB_TAPE_REGISTER(tb_head_prep_keyed_bf16)
 TB_TAPE_REGISTER(tb_head_prep_f32)
 TB_TAPE_REGISTER(tb_head_prep_bf16)

@@ -6,6 +6,7 @@
 //   u   <- N(u; post_w, post_b, post_eps, post_center)          when post_w is given
 //   v    = x[r] + u                 float;  written back to x[r] when rows is null and there was a u
 //   y[i] = N(v; w, b, eps, center)  one rounding to T;  w null: y[i] = v;  y null: nothing
+// or, for blocks that norm the stream itself, v = alpha x[r] + u, y[r] = N(v) and x[r] = y[r] before the rounding.
 //
 //   N(a; w, b, eps, center) = (a - m) / sqrt(mean((a - m)^2) + eps) * w + b,   m = center ? mean(a) : 0,  b may be null
 //
@@ -27,6 +28,17 @@ struct LayerNormTail {
     int E, k, rule;         // rule: RouterRule::scored
 };
 
+// Another thing that may ride along, for any number of rows: the experts that a table gives each row's token, with
+// equal weights, and the weight of an expert that every token passes, sigmoid(gate_w . row as stored).
+struct LayerNormPick {
+    const int* tok;         // [rows] token ids, or null: none of this
+    const int* table;       // [vocab, k]
+    const void* gate_w;     // [d] in the activations' type, or null: no such expert
+    int* idx;               // [rows, k]
+    float* wts;             // [rows, k], or [rows, k + 1] with gate_w
+    int k;
+};
+
 struct LayerNormArgs {
     float* x;
     const void* delta;
@@ -46,6 +58,9 @@ struct LayerNormArgs {
     void* y;
     int d;
     LayerNormTail tail;
+    float alpha = 1.f;      // the stream is multiplied by it before the sum
+    int replace = 0;        // 1: y becomes the stream itself (float, unrounded)
+    LayerNormPick pick = {nullptr, nullptr, nullptr, nullptr, nullptr, 0};
 };
 
 // Two partial statistics (count, mean, sum of squared deviations from that mean) joined into one: exact however
@@ -137,6 +152,24 @@ template <typename T, bool VEC> __device__ __forceinline__ void ln_store(T* p, c
     else stf(p, f[0]);
 }
 
+// a value as it comes back from the activations' type
+template <typename T> __device__ __forceinline__ float ln_rounded(float v) {
+    T t;
+    stf(&t, v);
+    return ldf(&t);
+}
+// row i's experts and weights; `dot` is this thread's part of gate_w . row
+__device__ __forceinline__ void ln_pick(const LayerNormPick& p, int i, float dot, float* red) {
+    const int kk = p.k + (p.gate_w ? 1 : 0);
+    for (int j = threadIdx.x; j < p.k; j += blockDim.x) {
+        p.idx[(size_t)i * p.k + j] = p.table[(size_t)p.tok[i] * p.k + j];
+        p.wts[(size_t)i * kk + j] = 1.0f / (float)p.k;
+    }
+    if (!p.gate_w) return;
+    const float z = block_sum(dot, red);
+    if (threadIdx.x == 0) p.wts[(size_t)i * kk + p.k] = 1.0f / (1.0f + expf(-z));
+}
+
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) post_add_layernorm_kernel(const LayerNormArgs a) {
     pdl_sync();
@@ -180,10 +213,10 @@ __global__ void __launch_bounds__(256) post_add_layernorm_kernel(const LayerNorm
             for (int e = 0; e < W; ++e) {
                 float u = ln_row[c + e];
                 if (a.post_w) u = (u - mean) * rstd * pw[e] + (a.post_b ? pb[e] : 0.f);
-                xv[e] += u;
+                xv[e] = a.alpha * xv[e] + u;
                 ln_row[c + e] = xv[e];
             }
-            if (!a.rows) ln_store<float, VEC>(xr + c, xv);
+            if (!a.rows && !a.replace) ln_store<float, VEC>(xr + c, xv);
         }
     } else {
         if (!a.y) return;
@@ -196,7 +229,7 @@ __global__ void __launch_bounds__(256) post_add_layernorm_kernel(const LayerNorm
     }
     if (!a.y) return;
     T* yr = static_cast<T*>(a.y) + (size_t)i * d;
-    float mean = 0.f, rstd = 1.f;
+    float mean = 0.f, rstd = 1.f, dot = 0.f;
     if (a.w) ln_stats<W>(ln_row, d, a.center != 0, a.eps, red, mean, rstd);
     for (int c = threadIdx.x * W; c < d; c += blockDim.x * W) {
         float o[W], w[W], b[W];
@@ -208,7 +241,15 @@ __global__ void __launch_bounds__(256) post_add_layernorm_kernel(const LayerNorm
             if (a.w) o[e] = (o[e] - mean) * rstd * w[e] + (a.b ? b[e] : 0.f);
         }
         ln_store<T, VEC>(yr + c, o);
+        if (a.replace) ln_store<float, VEC>(xr + c, o);
+        if (a.pick.gate_w) {
+            float gw[W];
+            ln_load<T, VEC>(static_cast<const T*>(a.pick.gate_w) + c, gw);
+#pragma unroll
+            for (int e = 0; e < W; ++e) dot += gw[e] * ln_rounded<T>(o[e]);
+        }
     }
+    if (a.pick.tok) ln_pick(a.pick, i, dot, red);
 }
 
 // The same with the row in registers: NCH pieces of eight entries a thread (widths that are multiples of eight up to
@@ -291,9 +332,9 @@ __global__ void __launch_bounds__(256) post_add_layernorm_reg_kernel(const Layer
             for (int e = 0; e < 8; ++e) {
                 float u = v[j][e];
                 if (a.post_w) u = (u - mean) * rstd * pw[e] + (a.post_b ? pb[e] : 0.f);
-                v[j][e] = xv[e] + u;
+                v[j][e] = a.alpha * xv[e] + u;
             }
-            if (!a.rows) store8(xr + c, v[j]);
+            if (!a.rows && !a.replace) store8(xr + c, v[j]);
         }
     } else {
         if (!a.y) return;
@@ -307,7 +348,7 @@ __global__ void __launch_bounds__(256) post_add_layernorm_reg_kernel(const Layer
     }
     if (!a.y) return;
     T* yr = static_cast<T*>(a.y) + (size_t)i * d;
-    float mean = 0.f, rstd = 1.f;
+    float mean = 0.f, rstd = 1.f, dot = 0.f;
     if (a.w) ln_stats_reg<NCH>(v, d, a.center != 0, a.eps, red, mean, rstd);
 #pragma unroll
     for (int j = 0; j < NCH; ++j) {
@@ -322,8 +363,16 @@ __global__ void __launch_bounds__(256) post_add_layernorm_reg_kernel(const Layer
             if (a.w) o[e] = (o[e] - mean) * rstd * w[e] + (a.b ? b[e] : 0.f);
         }
         store8(yr + c, o);
+        if (a.replace) store8(xr + c, o);
+        if (a.pick.gate_w) {
+            float gw[8];
+            load8(static_cast<const T*>(a.pick.gate_w) + c, gw);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) dot += gw[e] * ln_rounded<T>(o[e]);
+        }
         if (TAIL) store8(reinterpret_cast<T*>(ln_tail_smem) + c, o);      // what the router reads: the row as stored
     }
+    if (a.pick.tok) ln_pick(a.pick, i, dot, red);
     if (!TAIL) return;
     __syncthreads();
     constexpr int EPL = Vec16<T>::N;
@@ -365,7 +414,7 @@ static int post_add_layernorm_launch(const LayerNormArgs& a, int n_out, cudaStre
     if (n_out == 0) return 0;
     const uintptr_t all = (uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.wy | (uintptr_t)a.post_w |
                           (uintptr_t)a.post_b | (uintptr_t)a.w | (uintptr_t)a.b | (uintptr_t)a.y;
-    const bool vec = a.d % 8 == 0 && (all & 15) == 0;
+    const bool vec = a.d % 8 == 0 && (all & 15) == 0 && ((uintptr_t)a.pick.gate_w & 15) == 0;
     if (a.tail.w) {
         // the form that also routes: a few rows, the row in registers, the row as stored and the logits in 40 KB
         const LayerNormTail& t = a.tail;
@@ -423,11 +472,31 @@ extern "C" {
                         center, y, d, LayerNormTail{router_w, route_bias, route_idx, route_w, E, route_k, rule}};     \
         return post_add_layernorm_launch<T>(a, n_out, s);                                                             \
     }
+// The stream itself is normed:  x[r] = y[r] = N(alpha x[r] + u; w, b, eps)  with the mean taken off, x in float and y
+// rounded once to T.  With `tok`: what rides along (see LayerNormPick).
+#define TB_RENEW_LAYERNORM(SFX, T)                                                                                    \
+    int tb_renew_layernorm_##SFX(float* x, const void* delta, const void* wy, const int* pair_row,                    \
+                                 const float* topk_w, int k, float alpha, const float* w, const float* b, float eps,  \
+                                 void* y, int n_out, int d, const int* tok, const int* table, const void* gate_w,     \
+                                 int* idx, float* wts, int pick_k, cudaStream_t s) {                                  \
+        if (!w || !y || (!delta && !wy)) return TB_ERR_ARG;                                                           \
+        if (tok && (!table || !idx || !wts || pick_k <= 0)) return TB_ERR_ARG;                                        \
+        LayerNormArgs a{x, delta, wy, pair_row, topk_w, k, nullptr, nullptr, 0.f, 0, nullptr, w, b, eps,              \
+                        1, y, d, LayerNormTail{nullptr, nullptr, nullptr, nullptr, 0, 0, 0}};                         \
+        a.alpha = alpha;                                                                                              \
+        a.replace = 1;                                                                                                \
+        if (tok) a.pick = LayerNormPick{tok, table, gate_w, idx, wts, pick_k};                                        \
+        return post_add_layernorm_launch<T>(a, n_out, s);                                                             \
+    }
+TB_RENEW_LAYERNORM(f32, float)
+TB_RENEW_LAYERNORM(bf16, __nv_bfloat16)
 TB_LAYERNORM(f32, float)
 TB_LAYERNORM(bf16, __nv_bfloat16)
 }
 
 #include "tape.h"
+TB_TAPE_REGISTER(tb_renew_layernorm_f32)
+TB_TAPE_REGISTER(tb_renew_layernorm_bf16)
 TB_TAPE_REGISTER(tb_post_add_layernorm_f32)
 TB_TAPE_REGISTER(tb_post_add_layernorm_bf16)
 TB_TAPE_REGISTER(tb_post_add_layernorm_router_f32)

@@ -45,10 +45,10 @@ _SIGNATURES: Dict[str, str] = {
     "tb_random_fill_f32": "plulf", "tb_random_fill_bf16": "plulf",
     "tb_embed_scaled_f32": "pppiif", "tb_embed_scaled_bf16": "pppiif",
     "tb_post_add_rmsnorm_f32": "pppppipfppfpii", "tb_post_add_rmsnorm_bf16": "pppppipfppfpii",
-    "tb_gemm_simt_glu_f32": "pppppliiiiiiiff", "tb_gemm_simt_glu_bf16": "pppppliiiiiiiff",
+    "tb_gemm_simt_glu_f32": "pppppliiiiiiiffi", "tb_gemm_simt_glu_bf16": "pppppliiiiiiiffi",
     "tb_gemm_simt_batched_f32": "pppllliiiiiii", "tb_gemm_simt_batched_bf16": "pppllliiiiiii",
-    "tb_gemm_skinny_glu_bf16": "pppppliiiiiiiipiiff",
-    "tb_gemm_tc_glu_bf16": "ppppiiiiiiiff",
+    "tb_gemm_skinny_glu_bf16": "pppppliiiiiiiipiiffi",
+    "tb_gemm_tc_glu_bf16": "ppppiiiiiiiffi",
     "tb_post_add_rmsnorm_router_f32": "pppppipfpfpppppiiiii", "tb_post_add_rmsnorm_router_bf16": "pppppipfpfpppppiiiii",
     "tb_add_rmsnorm_router_scored_f32": "pppppippfpppppiiii", "tb_add_rmsnorm_router_scored_bf16": "pppppippfpppppiiii",
     "tb_router_rows_scored_bf16": "pppppppppiiii",
@@ -56,7 +56,7 @@ _SIGNATURES: Dict[str, str] = {
     "tb_moe_identity_rows_f32": "pppppiiii", "tb_moe_identity_rows_bf16": "pppppiiii",
     "tb_mlstm_scan_f32": "pppppppiiiiiff", "tb_mlstm_scan_bf16": "pppppppiiiiiff",
     "tb_mlstm_chunk_f32": "pppppppiiiiiff", "tb_mlstm_chunk_bf16": "pppppppiiiiiff",
-    "tb_mlstm_out_f32": "ppippiiifi", "tb_mlstm_out_bf16": "ppippiiifi",
+    "tb_mlstm_out_f32": "ppippiiifii", "tb_mlstm_out_bf16": "ppippiiifii",
     "tb_latent_prep_f32": "pippfpppppippiiiii", "tb_latent_prep_bf16": "pippfpppppippiiiii",
     "tb_latent_attention_mma_bf16": "ppppppppppppiiiiiiiiiiifppi",
     "tb_latent_attention_f32": "pppppppppppiiiiiiiiiifppi", "tb_latent_attention_bf16": "pppppppppppiiiiiiiiiifppi",
@@ -78,6 +78,17 @@ _SIGNATURES: Dict[str, str] = {
     "tb_moe_scaled_rows_f32": "ppppiii", "tb_moe_scaled_rows_bf16": "ppppiii",
     "tb_relu2_f32": "pl", "tb_relu2_bf16": "pl",
     "tb_post_add_layernorm_f32": "pppppippfipppfipii", "tb_post_add_layernorm_bf16": "pppppippfipppfipii",
+    "tb_renew_layernorm_f32": "pppppifppfpiipppppi", "tb_renew_layernorm_bf16": "pppppifppfpiipppppi",
+    "tb_moe_dispatch_shared": "ppppiii",
+    "tb_moe_terms_f32": "pppppppiii", "tb_moe_terms_bf16": "pppppppiii",
+    "tb_head_prep_keyed_f32": "pipifpppppppppiiiiii", "tb_head_prep_keyed_bf16": "pipifpppppppppiiiiii",
+    "tb_attention_window_heads_f32": "pppppppppppiiiiiiiiiiiiffipppifi",
+    "tb_attention_window_heads_bf16": "pppppppppppiiiiiiiiiiiiffipppifi",
+    "tb_attention_window_mma_heads_bf16": "pppppppppppiiiiiiiiiiiiffipppifi",
+    "tb_shift_mix_f32": "pppllpppipppii", "tb_shift_mix_bf16": "pppllpppipppii",
+    "tb_decay_prep_f32": "ppipppppiiii", "tb_decay_prep_bf16": "ppipppppiiii",
+    "tb_decay_scan_f32": "ppplppippiiii", "tb_decay_scan_bf16": "ppplppippiiii",
+    "tb_decay_step_f32": "ppipippppfplpippiiiii", "tb_decay_step_bf16": "ppipippppfplpippiiiii",
     "tb_post_add_layernorm_router_f32": "pppppippfipppfipiippppiii",
     "tb_post_add_layernorm_router_bf16": "pppppippfipppfipiippppiii",
 }
@@ -100,7 +111,8 @@ class TapeMap(ctypes.Structure):
     _fields_ = [("base", ctypes.c_ulonglong), ("size", ctypes.c_ulonglong), ("delta", ctypes.c_longlong)]
 
 
-_NO_STREAM = {"tb_attention_window_mma_tile_tokens": "ii", "tb_delta_state_size": "iiiii", "tb_delta_record_size": "i", "tb_delta_scan_lanes": "i", "tb_delta_value_pitch": "i", "tb_mlstm_state_size": "ii", "tb_latent_attention_tile_tokens": "i", "tb_attention_tile_tokens": "ii", "tb_gemm_tc_status": "", "tb_attention_prefill_tile_tokens": "",
+_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i", "tb_decay_value_pitch": "i", "tb_decay_scan_lanes": "i",
+              "tb_attention_window_mma_tile_tokens": "ii", "tb_delta_state_size": "iiiii", "tb_delta_record_size": "i", "tb_delta_scan_lanes": "i", "tb_delta_value_pitch": "i", "tb_mlstm_state_size": "ii", "tb_latent_attention_tile_tokens": "i", "tb_attention_tile_tokens": "ii", "tb_gemm_tc_status": "", "tb_attention_prefill_tile_tokens": "",
               "tb_attention_tc_tile_tokens": ""}
 
 _lock = threading.Lock()
@@ -402,6 +414,21 @@ def delta_record_size(dim: int) -> int:
 def delta_value_pitch(vdim: int) -> int:
     """Floats of a (token, head) row of values between the delta rule's two kernels."""
     return library().tb_delta_value_pitch(vdim)
+
+
+def decay_state_size(heads: int, dim: int, width: int) -> int:
+    """Floats of state that the decaying linear memory keeps per sequence (the heads' memories, then the last input)."""
+    return library().tb_decay_state_size(heads, dim, width)
+
+
+def decay_record_size(dim: int) -> int:
+    """Floats of the record that the decaying memory's first kernel leaves the scan per (token, head)."""
+    return library().tb_decay_record_size(dim)
+
+
+def decay_value_pitch(dim: int) -> int:
+    """Floats of a (token, head) row of values between the decaying memory's two kernels for prompts."""
+    return library().tb_decay_value_pitch(dim)
 
 
 def attention_window_mma_tile_tokens(nh: int, nkvh: int) -> int:

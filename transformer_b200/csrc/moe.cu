@@ -16,7 +16,7 @@
 //   w_j = exp(v_j - v_0) / sum_kept exp(v_i - v_0)    softmax over the kept logits (compute.rs:383-392)
 // topk_idx / topk_w are in descending-logit order.
 __device__ void dispatch_lists(const int* topk_idx, int* __restrict__ group_offsets, int* __restrict__ sorted_token,
-                               int* __restrict__ pair_row, int M, int k, int E, int* count, int* cursor);
+                               int* __restrict__ pair_row, int M, int k, int E, int* count, int* cursor, int pitch = 0);
 
 // With `lists` set, the block that finishes last (counted in lists.done, which it leaves at zero again) also
 // builds the dispatch lists from every token's choice: one kernel less between the router and the experts.
@@ -233,11 +233,13 @@ router_rows_kernel(const __nv_bfloat16* __restrict__ x1, const __nv_bfloat16* __
 // One block builds the dispatch lists for M = nt * k (token, choice) pairs:
 //   group_offsets[e] .. group_offsets[e+1]   rows of expert e in the sorted order
 //   sorted_token[r]                          token whose activation row r reads
-//   pair_row[t * k + j]                      row r that holds the pair's result
+//   pair_row[t * k + j]                      row r that holds the pair's result (t * pitch + j with a pitch above k;
+//                                            entry k is then row M + t, an expert that every token passes)
 // The order of the rows inside one expert is not fixed; no result depends on it (every row of a
 // product is computed alone, and the combine reads rows through pair_row in the order of j).
 __device__ void dispatch_lists(const int* topk_idx, int* __restrict__ group_offsets, int* __restrict__ sorted_token,
-                               int* __restrict__ pair_row, int M, int k, int E, int* count, int* cursor) {
+                               int* __restrict__ pair_row, int M, int k, int E, int* count, int* cursor, int pitch) {
+    if (pitch == 0) pitch = k;
     // One block, two passes over the pairs, and what they cost is the latency of reading each pair's expert: the
     // reads of eight rounds are asked for together, before any of them is used (a prompt of 2,048 tokens is eight
     // rounds of a 1,024-thread block: 9 -> 5 us for this kernel, which nothing runs beside).
@@ -280,19 +282,22 @@ __device__ void dispatch_lists(const int* topk_idx, int* __restrict__ group_offs
             if (ex[u] >= 0) {
                 const int r = atomicAdd(&cursor[ex[u]], 1);
                 sorted_token[r] = p / k;
-                pair_row[p] = r;
+                if (pitch == k) pair_row[p] = r;
+                else pair_row[p / k * pitch + p % k] = r;
             }
         }
     }
+    if (pitch > k)      // one more row per token, behind the experts' rows
+        for (int t = threadIdx.x; t < M / k; t += blockDim.x) pair_row[t * pitch + k] = M + t;
 }
 
 __global__ void __launch_bounds__(1024)
 moe_dispatch_kernel(const int* __restrict__ topk_idx, int* __restrict__ group_offsets,
-                    int* __restrict__ sorted_token, int* __restrict__ pair_row, int M, int k, int E) {
+                    int* __restrict__ sorted_token, int* __restrict__ pair_row, int M, int k, int E, int pitch) {
     pdl_sync();
     __shared__ int count[ROUTER_MAX_E + 1];
     __shared__ int cursor[ROUTER_MAX_E];
-    dispatch_lists(topk_idx, group_offsets, sorted_token, pair_row, M, k, E, count, cursor);
+    dispatch_lists(topk_idx, group_offsets, sorted_token, pair_row, M, k, E, count, cursor, pitch);
 }
 
 // delta[t, :] = sum_j w[t, j] * y[pair_row[t, j], :]   in float, j ascending = descending logit,
@@ -389,6 +394,33 @@ static int scaled_rows_launch(const void* x1, const float* topk_w, const int* pa
     if (M == 0) return 0;
     const int vec = d % 8 == 0 && (((uintptr_t)x1 | (uintptr_t)out) & 15) == 0;
     TB_LAUNCH((moe_scaled_rows_kernel<T>), M, 128, 0, s, (const T*)x1, topk_w, pair_row, (T*)out, d, k, vec);
+    return tb_last_error();
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) moe_terms_kernel(const T* __restrict__ x1, const T* __restrict__ gate_w,
+                                                        const int* __restrict__ tok, const int* __restrict__ table,
+                                                        const float* __restrict__ w_in, int* __restrict__ idx,
+                                                        float* __restrict__ wts, int d, int k) {
+    pdl_sync();
+    __shared__ float red[33];
+    const int t = blockIdx.x, kk = k + (gate_w ? 1 : 0);
+    for (int j = threadIdx.x; j < k; j += blockDim.x) {
+        if (table) idx[(size_t)t * k + j] = table[(size_t)tok[t] * k + j];
+        wts[(size_t)t * kk + j] = table ? 1.0f / (float)k : w_in[(size_t)t * k + j];
+    }
+    if (!gate_w) return;
+    float dot = 0.f;
+    for (int c = threadIdx.x; c < d; c += blockDim.x) dot += ldf(x1 + (size_t)t * d + c) * ldf(gate_w + c);
+    dot = block_sum(dot, red);
+    if (threadIdx.x == 0) wts[(size_t)t * kk + k] = 1.0f / (1.0f + expf(-dot));
+}
+template <typename T>
+static int moe_terms_launch(const void* x1, const void* gate_w, const int* tok, const int* table, const float* w_in,
+                            int* idx, float* wts, int nt, int d, int k, cudaStream_t s) {
+    if (nt < 0 || d <= 0 || k <= 0 || !wts || (table ? (!tok || !idx) : !w_in)) return TB_ERR_ARG;
+    if (nt == 0) return 0;
+    TB_LAUNCH((moe_terms_kernel<T>), nt, 128, 0, s, (const T*)x1, (const T*)gate_w, tok, table, w_in, idx, wts, d, k);
     return tb_last_error();
 }
 
@@ -504,8 +536,28 @@ int tb_moe_dispatch(const int* topk_idx, int* group_offsets, int* sorted_token, 
                     cudaStream_t s) {
     if (M < 0 || k <= 0 || E <= 0) return TB_ERR_ARG;
     if (E > ROUTER_MAX_E) return TB_ERR_UNSUPPORTED;
-    TB_LAUNCH((moe_dispatch_kernel), 1, 1024, 0, s, topk_idx, group_offsets, sorted_token, pair_row, M, k, E);
+    TB_LAUNCH((moe_dispatch_kernel), 1, 1024, 0, s, topk_idx, group_offsets, sorted_token, pair_row, M, k, E, 0);
     return tb_last_error();
+}
+// The same for tokens that also pass an expert of their own besides: pair_row has k + 1 entries a token, the last of
+// them row M + t.
+int tb_moe_dispatch_shared(const int* topk_idx, int* group_offsets, int* sorted_token, int* pair_row, int M, int k,
+                           int E, cudaStream_t s) {
+    if (M < 0 || k <= 0 || E <= 0 || M % k) return TB_ERR_ARG;
+    if (E > ROUTER_MAX_E) return TB_ERR_UNSUPPORTED;
+    TB_LAUNCH((moe_dispatch_kernel), 1, 1024, 0, s, topk_idx, group_offsets, sorted_token, pair_row, M, k, E, k + 1);
+    return tb_last_error();
+}
+// The terms of every token's sum over experts where the choice does not come from a router's kernel alone:
+//   table (may be null): idx[t, j] = table[tok[t], j], every weight 1 / k;  w_in [nt, k]: the weights of a choice made
+//   elsewhere;  gate_w (may be null): wts has k + 1 entries a token, the last sigmoid(gate_w . x1[t]).
+int tb_moe_terms_f32(const void* x1, const void* gate_w, const int* tok, const int* table, const float* w_in, int* idx,
+                     float* wts, int nt, int d, int k, cudaStream_t s) {
+    return moe_terms_launch<float>(x1, gate_w, tok, table, w_in, idx, wts, nt, d, k, s);
+}
+int tb_moe_terms_bf16(const void* x1, const void* gate_w, const int* tok, const int* table, const float* w_in, int* idx,
+                      float* wts, int nt, int d, int k, cudaStream_t s) {
+    return moe_terms_launch<__nv_bfloat16>(x1, gate_w, tok, table, w_in, idx, wts, nt, d, k, s);
 }
 int tb_moe_combine_f32(const void* y, const int* pair_row, const float* topk_w, void* delta, int nt, int d, int k,
                        cudaStream_t s) {
@@ -533,5 +585,8 @@ TB_TAPE_REGISTER(tb_moe_scaled_rows_bf16)
 TB_TAPE_REGISTER(tb_moe_identity_rows_f32)
 TB_TAPE_REGISTER(tb_moe_identity_rows_bf16)
 TB_TAPE_REGISTER(tb_moe_dispatch)
+TB_TAPE_REGISTER(tb_moe_dispatch_shared)
+TB_TAPE_REGISTER(tb_moe_terms_f32)
+TB_TAPE_REGISTER(tb_moe_terms_bf16)
 TB_TAPE_REGISTER(tb_moe_combine_f32)
 TB_TAPE_REGISTER(tb_moe_combine_bf16)

@@ -21,7 +21,7 @@ from ..cache.paged import Cache
 from ..cache.slots import CacheError
 from ..csrc import lib
 from ..parts.block import build_layer, resolve
-from ..parts.base import EMBEDDINGS, HEADS, JOINTS, NORMS, NormedDelta, PairDelta
+from ..parts.base import EMBEDDINGS, HEADS, JOINTS, NORMS, NormedDelta, PairDelta, StreamRows
 from ..parts.spec import ModelSpec
 from .context import StepContext, Workspace, weak_callback
 from .tape import LayerTape, moves, run_tensors
@@ -38,6 +38,8 @@ def _pending_signature(pending):
         return None
     if isinstance(pending, torch.Tensor):
         return ("t", pending.data_ptr(), tuple(pending.shape))
+    if isinstance(pending, StreamRows):
+        return ("s", pending.rows.data_ptr(), tuple(pending.rows.shape))
     if isinstance(pending, PairDelta):
         return ("p", _pending_signature(pending.first), _pending_signature(pending.second))
     if isinstance(pending, NormedDelta):      # names a weight of the layer before: equal only for the same layer

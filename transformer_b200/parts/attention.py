@@ -29,6 +29,14 @@ learned number l, weights ``vmix``).  With any of these the kernel between the p
 at once.  That kernel turns adjacent pairs; a rotary part that pairs entry i with i + dims/2 is met by reordering,
 once at binding, the rows of the query and key projections (and of their norm weights and convolutions) that make the
 rotated entries: a permutation applied to queries and keys alike, which leaves every score as it was.
+
+A third family: heads whose values are their keys as projected (``values`` = "keys": no value projection; the value
+cache holds the key before norm and rotation).  With it: biases on the query and key projections (``bias``, weights
+``bqk``); an RMS norm per head without weights (``qk_norm="unit"``, ``eps``); one sigmoid gate per head on the output
+(``head_gate``; its rows ride in the merged product); a fixed number that joins the softmax's denominator as
+exp(sink_value) (``sink_value``); a multiplier of the output (``out_scale``).  The kernel between the product and the
+attention is ``tb_head_prep_keyed``; the attention is the windowed one.  This family can leave its heads' outputs in a
+wider row (``forward_rows``) for a mixer that stands beside it.
 """
 from __future__ import annotations
 
@@ -52,7 +60,7 @@ USE_WINDOW_MMA = True   # the windowed path, bfloat16: the tensor-core kernel be
 @MIXERS.register("attention")
 class Attention(Mixer):
     """params: width, nh, nkvh, dh, position (a PartSpec of a rotary encoding, or None); optional: dv, scale, softcap,
-    window, keep_first, qk_norm, eps, gate (see the head of this file)."""
+    window, keep_first, qk_norm, eps, gate and the further families' (see the head of this file)."""
 
     def __init__(self, params, dtype, device):
         super().__init__(params, dtype, device)
@@ -73,7 +81,7 @@ class Attention(Mixer):
         self.qk_norm = params.get("qk_norm")
         self.gate = bool(params.get("gate", False))
         self.eps = float(params.get("eps", 0.0))
-        if self.qk_norm not in (None, "whole", "head"):
+        if self.qk_norm not in (None, "whole", "head", "unit"):
             raise ValueError(f"unknown query/key norm {self.qk_norm!r}")
         self.conv_taps = int(params.get("conv_taps") or 0)          # 0: no convolution on the projections
         self.temperature = bool(params.get("temperature", False))
@@ -85,16 +93,30 @@ class Attention(Mixer):
             raise ValueError(f"value_mix is 'source', 'blend' or absent, got {self.value_mix!r}")
         if self.conv_taps < 0 or self.conv_taps > 16 or self.chunk < 0:
             raise ValueError("convolutions of 1 to 16 taps; chunk not negative")
+        # the third family: values that are the keys
+        if params.get("values", "own") not in ("own", "keys"):
+            raise ValueError(f"values are 'own' or 'keys', got {params.get('values')!r}")
+        self.keyed = params.get("values", "own") == "keys"
+        self.bias = bool(params.get("bias", False))
+        self.head_gate = bool(params.get("head_gate", False))
+        self.out_scale = float(params.get("out_scale", 1.0))
+        self.sink_value = params.get("sink_value")
+        if not self.keyed and (self.bias or self.head_gate or self.out_scale != 1.0 or self.sink_value is not None or
+                               self.qk_norm == "unit"):
+            raise ValueError("biases, a gate per head, a fixed sink, an output multiplier and a norm without weights go "
+                             "with values that are the keys")
         # the second family of mechanisms: its own kernel between the product and the attention
         self.prepared = bool(self.conv_taps or self.qk_norm == "head" or self.temperature or self.value_rotation or
                              self.value_mix)
         if self.prepared and (self.gate or self.qk_norm == "whole"):
             raise ValueError("a norm over the whole projection or an output gate does not go with the per-head family")
+        if self.keyed and (self.prepared or self.gate or self.sink or self.qk_norm == "whole" or self.dv != self.dh):
+            raise ValueError("values that are the keys go with the parameters of their own family, a window, a chunk and a cap")
         if self.dv <= 0 or self.dv > 256 or self.window < 0 or self.keep_first < 0 or self.softcap < 0:
             raise ValueError("value heads of 1..256 entries; window, keep_first and softcap not negative")
         # any of the further mechanisms takes the step to the windowed kernels
         self.extended = bool(self.dv != self.dh or self.softcap or self.window or self.qk_norm or self.gate or
-                             "scale" in params or self.prepared or self.chunk or self.sink)
+                             "scale" in params or self.prepared or self.chunk or self.sink or self.keyed)
         if not self.extended and (self.dh % 16):
             raise ValueError(f"the attention kernels take head sizes 16, 32, ..., 256; got {self.dh}")
         self.rdims = 0
@@ -104,6 +126,8 @@ class Attention(Mixer):
             self.rdims = int(pos.get()["dh"])
             if self.rdims > self.dh:
                 raise ValueError(f"a rotation of {self.rdims} entries does not fit heads of {self.dh}")
+        if self.keyed and isinstance(pos, PartSpec) and pos.get().get("pairing", "adjacent") != "adjacent":
+            raise ValueError("values that are the keys take a rotation of adjacent pairs")
         self.value_position = None
         if self.value_rotation:
             if self.dv % 2 or not isinstance(pos, PartSpec):
@@ -112,6 +136,10 @@ class Attention(Mixer):
             self.value_position = POSITIONS.build(PartSpec.of("rope", dh=self.dv, theta=pp["theta"], pairing="adjacent",
                                                               positions=pp["positions"]), dtype, device)
         self.qkv_width = (self.nh + self.nkvh) * self.dh + self.nkvh * self.dv + (self.nh * self.dv if self.gate else 0)
+        if self.keyed:      # q | k | one gate per head; the bound weight gets rows of zeros up to a multiple of eight
+            self.proj_rows = (self.nh + self.nkvh) * self.dh + (self.nh if self.head_gate else 0)
+            self.qkv_width = (self.proj_rows + 7) // 8 * 8
+            self.rows_width = self.nh * self.dh
         self.scale = float(params["scale"]) if "scale" in params else 1.0 / math.sqrt(self.dh)
         # query tiles this mixer asks the step to plan: the general kernel's, and the prompt kernel's
         self.general_tile = lib.attention_tile_tokens(self.nh, self.nkvh)
@@ -135,7 +163,7 @@ class Attention(Mixer):
 
     def parameters(self):
         decl = {
-            "wqkv": ParamDecl((self.qkv_width, self.d)),
+            "wqkv": ParamDecl((self.proj_rows if self.keyed else self.qkv_width, self.d)),
             "wo": ParamDecl((self.d, self.nh * self.dv)),
         }
         if self.qk_norm == "whole":
@@ -144,6 +172,8 @@ class Attention(Mixer):
         elif self.qk_norm == "head":
             decl["q_norm"] = ParamDecl((self.dh,), "norm", "ones")
             decl["k_norm"] = ParamDecl((self.dh,), "norm", "ones")
+        if self.bias:
+            decl["bqk"] = ParamDecl(((self.nh + self.nkvh) * self.dh,), "norm", "normal")
         if self.conv_taps:
             decl["conv"] = ParamDecl((self.qkv_width, self.conv_taps), "norm", "normal")
         if self.temperature:
@@ -160,6 +190,12 @@ class Attention(Mixer):
         super().bind(tensors)
         if self.position is not None:
             self.position.bind({n: tensors["position." + n] for n in self.position.parameters()})
+        if self.keyed:
+            w = self.weights["wqkv"]
+            if self.qkv_width != self.proj_rows:
+                self.weights["wqkv"] = torch.cat([w, w.new_zeros((self.qkv_width - self.proj_rows, self.d))]).contiguous()
+            if self.sink_value is not None:
+                self.weights["sink"] = torch.full((self.nh,), float(self.sink_value), dtype=torch.float32, device=w.device)
         if "vmix" in self.weights:
             self.weights["vmix"] = self.weights["vmix"].float().reshape(1).contiguous()
         if self.prepared and self.rdims and self.position.rotation()[2]:
@@ -246,7 +282,35 @@ class Attention(Mixer):
                              sinks=w.get("sink") if self.sink else None)
         matmul_nt(o, w["wo"], out)
 
+    def forward_rows(self, ctx, x1, rows, cache, state) -> None:
+        """The heads' outputs, gated and scaled, for the family whose values are the keys."""
+        if not self.keyed:
+            raise NotImplementedError("only attention whose values are the keys leaves its rows to another part's product")
+        nt = x1.shape[0]
+        w = self.weights
+        z = ctx.scratch("attn.qkv", (nt, self.qkv_width), self.dtype)        # q | k | gate per head | padding
+        matmul_nt(x1, w["wqkv"], z)
+        table = ctx.page_table(cache)
+        cos = sin = None
+        if self.rdims:
+            cos, sin, _ = self.position.rotation()
+        kc, vc = (cache.k, cache.v) if cache.writable else (None, None)
+        q = ctx.scratch("attn.q", (nt, self.nh * self.dh), self.dtype)
+        lib.call("tb_head_prep_keyed_" + lib.suffix(self.dtype), lib.ptr(z), self.qkv_width, lib.ptr(w.get("bqk")),
+                 1 if self.qk_norm == "unit" else 0, self.eps, lib.ptr(cos), lib.ptr(sin), lib.ptr(q), lib.ptr(kc),
+                 lib.ptr(vc), lib.ptr(ctx.tok_seq), lib.ptr(ctx.tok_pos), lib.ptr(ctx.seq_start), lib.ptr(table),
+                 ctx.max_pages, nt, self.nh, self.nkvh, self.dh, self.rdims)
+        gate = z[:, (self.nh + self.nkvh) * self.dh:] if self.head_gate else None
+        run_window_attention(ctx, self, q, rows, gate, cache, table, nt, self.window if self.window else 1 << 30,
+                             q_stride=self.nh * self.dh, sinks=w.get("sink"),
+                             heads=(1 if self.head_gate else 0, self.out_scale, rows.stride(0)))
+
     def forward(self, ctx, x1, out, cache, state) -> None:
+        if self.keyed:
+            rows = ctx.scratch("attn.o", (x1.shape[0], self.rows_width), self.dtype)
+            self.forward_rows(ctx, x1, rows, cache, state)
+            matmul_nt(rows, self.weights["wo"], out)
+            return
         if self.prepared:
             self._forward_prepared(ctx, x1, out, cache, state)
             return
@@ -355,9 +419,11 @@ class Attention(Mixer):
 
 
 def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=None, sinks=None, ocos=None,
-                         osin=None) -> None:
+                         osin=None, heads=None) -> None:
     """The windowed attention of the step's rotated queries ``z`` over the cache, into ``o`` (gate applied).
-    ``sinks``: a number per head in the softmax's denominator; ``ocos, osin``: tables that turn the output back."""
+    ``sinks``: a number per head in the softmax's denominator; ``ocos, osin``: tables that turn the output back;
+    ``heads`` = (gate holds one number per head, output multiplier, pitch of ``o``)."""
+    which, more = ("", ()) if heads is None else ("_heads", heads)
     sfx = lib.suffix(m.dtype)
     q_stride = m.qkv_width if q_stride is None else q_stride
     if m.window_tile and USE_WINDOW_MMA:
@@ -368,11 +434,11 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
         pages = (reach + m.keep_first + 63) // 64 + 2
         splits = int(max(1, min(16, pages, (2 * ctx.engine.sm_count) // max(1, tiles.count * m.nkvh))))
         partial = ctx.scratch("attn.partial", (nt, m.nh, splits, m.dv + 2), torch.float32) if splits > 1 else None
-        if lib.try_call("tb_attention_window_mma_bf16", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v),
+        if lib.try_call(f"tb_attention_window_mma{which}_bf16", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v),
                         lib.ptr(gate), lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos),
                         lib.ptr(table), lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width,
                         m.nh, m.nkvh, m.dh, m.dv, splits, window, m.keep_first, m.scale, m.softcap, m.chunk,
-                        lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin)):
+                        lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin), *more):
             return
     tiles = ctx.tiles(m.general_tile)
     # slices of the visited keys so that a few sequences still fill the GPU: a function of the batch's shape alone (a
@@ -381,7 +447,7 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
     reach = min(window, 1 << 20) if not m.chunk else min(window, m.chunk)
     splits = int(max(1, min(splits, (reach + m.keep_first + 31) // 32 + 1)))
     partial = ctx.scratch("attn.partial", (nt, m.nh, splits, m.dv + 2), torch.float32) if splits > 1 else None
-    lib.call("tb_attention_window_" + sfx, lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v), lib.ptr(gate),
+    lib.call(f"tb_attention_window{which}_{sfx}", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v), lib.ptr(gate),
              lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos), lib.ptr(table),
              lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width, m.nh, m.nkvh, m.dh, m.dv,
-             splits, window, m.keep_first, m.scale, m.softcap, m.chunk, lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin))
+             splits, window, m.keep_first, m.scale, m.softcap, m.chunk, lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin), *more)

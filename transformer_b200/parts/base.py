@@ -53,7 +53,7 @@ import torch
 class ParamDecl:
     shape: Tuple[int, ...]
     role: str = "matrix"     # "matrix" | "norm" | "table"
-    init: str = "normal"     # "normal" | "ones"
+    init: str = "normal"     # "normal" | "ones" | "distinct:n" (a table: integers below n, those of a row differing)
 
 
 @dataclass(frozen=True)
@@ -112,6 +112,13 @@ class NormedDelta:
     center: bool = False
 
 
+@dataclass
+class StreamRows:
+    """Nothing is left to be added to the stream, and the stream's rows, rounded to the activation type, already lie in
+    ``rows``: left by a block whose last kernel norms the stream itself, for a block that reads it as it is."""
+    rows: torch.Tensor        # [nt, d]
+
+
 class Part:
     graph_safe = False      # see the head of this file; the parts of this package set it
     launches_only = False   # all device work goes through csrc.lib launchers (or reports itself with lib.foreign):
@@ -146,7 +153,8 @@ class NormTail:
     the same kernel (the rows are at hand there; a kernel of its own would wait for them and read them back).
     ``kind`` names it; a norm lists the kinds it can do in ``Norm.tails`` and is handed nothing else.
     "router": ``weights`` [E, d], ``k``; the norm fills ``index`` [rows, k] (int32) and ``scores`` [rows, k] (float)
-    with each row's k experts and their softmax weights, by the rules of the router kernel."""
+    with each row's k experts and their softmax weights, by the rules of the router kernel.
+    "terms": the experts that ``table`` gives the row's token, and what ``gate`` gives an expert besides."""
     kind: str
     weights: Any = None
     k: int = 0
@@ -155,6 +163,9 @@ class NormTail:
     scored: bool = False     # "router": softmax over all outputs, choice by score + bias, weights = the chosen scores
     bias: Any = None
     sigmoid: bool = False    # "router": the k largest logits, weights = their sigmoids as they are
+    table: Any = None        # "terms": [vocab, k] int32, the experts of every token id, each with weight 1 / k
+    gate: Any = None         # "terms": [d], the gate of an expert that every token passes; ``scores`` is then [rows, k + 1],
+                             #          the last entry sigmoid(gate . row)
 
     @property
     def rule(self) -> int:
@@ -168,12 +179,20 @@ class Norm(Part):
     takes_pair_delta = False
     can_warm = False           # forward takes ``warm=``: a weight of the next part to fetch into L2 meanwhile
     tails: tuple = ()          # kinds of NormTail that forward(..., tail=) computes along the way
+    renew_tails: tuple = ()    # the same for renew(..., tail=)
 
     def forward(self, ctx, x, delta, rows, y) -> None:
         raise NotImplementedError
 
+    def renew(self, ctx, x, delta, y, tail=None) -> None:
+        """x <- y = norm(stream * x + delta), x in float, y rounded to the activation type; ``stream`` is the norm's own
+        parameter.  For blocks that norm the stream itself (optional)."""
+        raise NotImplementedError
+
 
 class Mixer(Part):
+    rows_width: Optional[int] = None    # the width of the rows that forward_rows leaves for the output product
+
     def cache_need(self) -> Optional[CacheNeed]:
         return None
 
@@ -181,6 +200,11 @@ class Mixer(Part):
         return None
 
     def forward(self, ctx, x1, out, cache, state) -> None:
+        raise NotImplementedError
+
+    def forward_rows(self, ctx, x1, rows, cache, state) -> None:
+        """What ``forward`` does up to its output product (weight "wo", [width, rows_width]): ``rows`` [nt, rows_width],
+        a view with a pitch, receives what that product reads.  For mixers that stand beside another one."""
         raise NotImplementedError
 
 

@@ -17,7 +17,8 @@ return value is what this block leaves.  A block that wants its sums done at onc
 """
 from __future__ import annotations
 
-from .base import ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, NormedDelta, PairDelta, WeightedRows
+from .base import ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, NormedDelta, PairDelta, StreamRows, WeightedRows
+from .spec import PartSpec
 
 
 def build_layer(spec, dtype, device):
@@ -248,9 +249,68 @@ class ParallelLayer:
         return PairDelta(out_m, out_f)
 
 
+@ARRANGEMENTS.register("post_norm")
+class PostNormLayer:
+    """A block that norms the stream itself behind each of its parts, which read the stream as it is:
+
+        x <- norm_m(alpha x + mixer(x));   x <- norm_f(alpha x + feed_forward(x))
+
+    ``alpha`` is the norms' own ``stream`` parameter; both must be of a kind that offers ``renew``.  A layer may have
+    no feed-forward.  One kernel does the scaled sum, the norm, the float stream and the rounded rows that the next part
+    reads (the experts' weighted sum on the way in, the experts' choice on the way out where it can ride along); the
+    block leaves those rows as a :class:`StreamRows`, so the block behind it starts with its mixer."""
+
+    def __init__(self, spec, dtype, device):
+        if spec.mixer_norm is None:
+            raise ValueError("the post_norm arrangement needs a norm behind the mixer")
+        self.spec = spec
+        # what a first block starts with: the stream as it is, rounded
+        self.read = NORMS.build(PartSpec.of("none", width=spec.mixer_norm.get()["width"]), dtype, device)
+        self.mixer = MIXERS.build(spec.mixer, dtype, device)
+        self.mixer_norm = NORMS.build(spec.mixer_norm, dtype, device)
+        self.feed_forward = self.feed_forward_norm = None
+        if spec.feed_forward is not None:
+            if spec.feed_forward_norm is None:
+                raise ValueError("a post_norm block with a feed-forward needs the norm behind it")
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, dtype, device)
+            self.feed_forward_norm = NORMS.build(spec.feed_forward_norm, dtype, device)
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(p.graph_safe for p in self.parts().values())
+
+    @property
+    def launches_only(self) -> bool:
+        return all(p.launches_only for p in self.parts().values())
+
+    def parts(self):
+        out = {"mixer": self.mixer, "mixer_norm": self.mixer_norm}
+        if self.feed_forward is not None:
+            out.update({"feed_forward": self.feed_forward, "feed_forward_norm": self.feed_forward_norm})
+        return out
+
+    def forward(self, ctx, x, pending, cache_view, state):
+        nt, d = x.shape
+        x1 = ctx.scratch("block.x1", (nt, d), ctx.dtype)
+        delta = ctx.scratch("block.delta", (nt, d), ctx.dtype)
+        if not isinstance(pending, StreamRows):
+            pending = resolve(pending, self.read, delta, x=x, ctx=ctx)
+            self.read.forward(ctx, x, pending, None, x1)
+        self.mixer.forward(ctx, x1, delta, cache_view, state)
+        tail = None if self.feed_forward is None else self.feed_forward.norm_tail(ctx, nt)
+        if tail is not None and tail.kind not in self.mixer_norm.renew_tails:
+            tail = None
+        self.mixer_norm.renew(ctx, x, delta, x1, tail=tail)
+        if self.feed_forward is not None:
+            lazy = self.feed_forward.forward(ctx, x1, delta) if tail is None else \
+                self.feed_forward.forward(ctx, x1, delta, tail=tail)
+            self.feed_forward_norm.renew(ctx, x, delta if lazy is None else lazy, x1)
+        return StreamRows(x1)
+
+
 def add_pending(ctx, x, pending) -> None:
     """x += pending, at once and in float, for an arrangement that does not leave the sum to a norm."""
-    if pending is None:
+    if pending is None or isinstance(pending, StreamRows):
         return
     if isinstance(pending, NormedDelta):
         from .norm import post_add_rmsnorm
@@ -271,6 +331,8 @@ def add_pending(ctx, x, pending) -> None:
 def resolve(pending, norm, into, x=None, ctx=None):
     """A pending WeightedRows stays as it is for a norm that sums it itself; else it is summed into ``into``.  A
     pending NormedDelta stays for a norm that takes one; else it is normed and added to the stream ``x`` now."""
+    if isinstance(pending, StreamRows):
+        return None
     if isinstance(pending, NormedDelta):
         if getattr(norm, "takes_normed_delta", False):
             return pending

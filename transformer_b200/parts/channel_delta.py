@@ -123,5 +123,5 @@ class ChannelDelta(Mixer):
                  lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, self.G, H, self.dim, self.vdim, self.taps)
         y = ctx.scratch("delta.y", (nt, self.hv), self.dtype)
         lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(gz), gz.stride(0), lib.ptr(w["norm"]), lib.ptr(y), nt, H,
-                 self.vdim, self.eps, 1 if self.gate_act == "silu" else 0)
+                 self.vdim, self.eps, 1 if self.gate_act == "silu" else 0, self.hv)
         matmul_nt(y, w["wo"], out)

@@ -26,7 +26,7 @@ class DenseSwiGLU(FeedForward):
     more column (and zeros up to a multiple of eight), and the kernel that applies the pair's biases and the
     activation writes a one into that column of ``h``.  ``glu_limit`` (with ``glu_alpha``, default 1): the pair
     becomes g' * sigmoid(alpha g') * (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit) instead of
-    silu(g) * u, in the product's epilogue."""
+    silu(g) * u, in the product's epilogue.  ``act`` = "gelu_tanh": gelu(g) * u with the tanh form of gelu, there too."""
     graph_safe = True
     launches_only = True
 
@@ -39,6 +39,13 @@ class DenseSwiGLU(FeedForward):
         self.glu = None if limit is None else (float(params.get("glu_alpha", 1.0)), float(limit))
         if self.glu is not None and self.bias:
             raise ValueError("the clamped pair has no form with biases")
+        act = params.get("act", "silu")
+        if act not in ("silu", linear.GELU_TANH):
+            raise ValueError(f"unknown activation {act!r}; this part has 'silu' and 'gelu_tanh'")
+        if act != "silu":
+            if self.glu is not None or self.bias:
+                raise ValueError("the tanh form of gelu goes with neither the clamped pair nor biases")
+            self.glu = act
 
     def parameters(self):
         decl = {"wgu": ParamDecl((2 * self.di, self.d)), "wd": ParamDecl((self.d, self.di))}
@@ -121,7 +128,12 @@ class MoE(FeedForward):
       to the lower index); the weights are the chosen scores as they are.
     * ``weight_on`` = "input": the weight multiplies what the expert reads, out = sum_e expert_e(w_e x1), instead of
       what it returns.  Every (token, choice) pair gets its own scaled copy of the token's row (one kernel, which
-      also puts the rows in the experts' order), the experts run on those, and their results are summed unweighted."""
+      also puts the rows in the experts' order), the experts run on those, and their results are summed unweighted.
+    * ``scoring`` = "table": no router.  A table (weight ``table``, [vocab, nexp_use] int32, the entries of a row differ)
+      gives every token id its experts; every weight is 1 / nexp_use.
+    * ``shared_di`` = n: one more expert of width n (weights ``shared_wgu``, ``shared_wd``; ``shared_limit`` and
+      ``glu_alpha`` as above), which every token passes; its result is multiplied by sigmoid(gate . x1), one number a
+      token (weight ``shared_gate``), and joins the same weighted sum."""
     graph_safe = True
     launches_only = True
 
@@ -138,7 +150,7 @@ class MoE(FeedForward):
         if self.R > 1024:
             raise ValueError(f"the routing kernels take up to 1024 experts, got {self.R}")
         self.scoring = params.get("scoring", "kept")
-        if self.scoring not in ("kept", "all", "sigmoid"):
+        if self.scoring not in ("kept", "all", "sigmoid", "table"):
             raise ValueError(f"unknown router scoring {self.scoring!r}")
         self.weight_on = params.get("weight_on", "output")
         if self.weight_on not in ("output", "input"):
@@ -151,16 +163,41 @@ class MoE(FeedForward):
         limit = params.get("glu_limit")
         self.glu = None if limit is None else (float(params.get("glu_alpha", 1.0)), float(limit))
         self.plain_router = self.scoring == "kept" and not self.identity
+        self.table = self.scoring == "table"
+        self.vocab = int(params.get("vocab", 0))
+        if self.table and (self.identity or self.weight_on == "input" or self.vocab <= 0):
+            raise ValueError("a table of experts needs 'vocab' and goes with neither pass-through experts nor weights on the input")
+        self.shared = int(params.get("shared_di") or 0)
+        if self.shared and (self.identity or self.weight_on == "input"):
+            raise ValueError("a shared expert goes with neither pass-through experts nor weights on the input")
+        limit = params.get("shared_limit")
+        self.shared_glu = None if limit is None else (float(params.get("glu_alpha", 1.0)), float(limit))
+        self.terms = self.k + (1 if self.shared else 0)       # of a token's sum
 
     def parameters(self):
         decl = {
-            "router": ParamDecl((self.R, self.d)),
             "wgu": ParamDecl((self.E, 2 * self.di, self.d)),
             "wd": ParamDecl((self.E, self.d, self.di)),
         }
+        if self.table:
+            decl["table"] = ParamDecl((self.vocab, self.k), "table", f"distinct:{self.E}")
+        else:
+            decl["router"] = ParamDecl((self.R, self.d))
+        if self.shared:
+            decl["shared_wgu"] = ParamDecl((2 * self.shared, self.d))
+            decl["shared_wd"] = ParamDecl((self.d, self.shared))
+            decl["shared_gate"] = ParamDecl((1, self.d))
         if self.correction:
             decl["correction"] = ParamDecl((self.R,), "norm", "normal")
         return decl
+
+    def bind(self, tensors) -> None:
+        super().bind(tensors)
+        if self.table:
+            t = self.weights["table"]
+            lo, hi = int(t.min()), int(t.max())
+            if lo < 0 or hi >= self.E:
+                raise ValueError(f"the table names experts {lo}..{hi}, but there are {self.E}")
 
     def early_weights(self):
         """The router's matrix: small, and every token's block waits for all of it."""
@@ -219,6 +256,11 @@ class MoE(FeedForward):
 
     def norm_tail(self, ctx, nt):
         """For a few tokens the router rides along with the norm before this part."""
+        if self.table:
+            return NormTail("terms", table=self.weights["table"], k=self.k,
+                            gate=self.weights["shared_gate"] if self.shared else None,
+                            index=ctx.scratch("moe.topk_idx", (nt, self.k), torch.int32),
+                            scores=ctx.scratch("moe.terms_w", (nt, self.terms), torch.float32))
         if nt > ROUTER_TAIL_ROWS:
             return None
         return NormTail("router", weights=self.weights["router"], k=self.k,
@@ -227,7 +269,59 @@ class MoE(FeedForward):
                         scored=self.scoring == "all", bias=self.weights.get("correction"),
                         sigmoid=self.scoring == "sigmoid")
 
+    def _terms(self, ctx, x1, tail):
+        """(experts [nt, k], weights [nt, terms]) of every token's sum, where a table chooses or a shared expert joins."""
+        nt = x1.shape[0]
+        if tail is not None and tail.kind == "terms":
+            return tail.index, tail.scores
+        table = self.weights.get("table")
+        if table is None:
+            idx, w_in = (tail.index, tail.scores) if tail is not None else self.route(ctx, x1)[:2]
+        else:
+            idx, w_in = ctx.scratch("moe.topk_idx", (nt, self.k), torch.int32), None
+        w = ctx.scratch("moe.terms_w", (nt, self.terms), torch.float32)
+        lib.call("tb_moe_terms_" + lib.suffix(self.dtype), lib.ptr(x1), lib.ptr(self.weights.get("shared_gate")),
+                 lib.ptr(ctx.tok_ids), lib.ptr(table), lib.ptr(w_in), lib.ptr(idx), lib.ptr(w), nt, self.d, self.k)
+        return idx, w
+
+    def _shared(self, ctx, x1, out) -> None:
+        h = ctx.scratch("moe.shared_h", (x1.shape[0], self.shared), self.dtype)
+        grouped_matmul(x1, self.weights["shared_wgu"], h, swiglu=True, glu=self.shared_glu)
+        matmul_nt(h, self.weights["shared_wd"], out)
+
+    def _forward_terms(self, ctx, x1, tail):
+        """The step where a table chooses the experts or a shared expert joins: the experts' rows and the shared
+        expert's lie one behind the other, and all of them are terms of one weighted sum."""
+        nt = x1.shape[0]
+        M = nt * self.k
+        rows = ctx.scratch("moe.y", (M + (nt if self.shared else 0), self.d), self.dtype)
+        y = rows[:M]
+        idx, w = self._terms(ctx, x1, tail)
+        ctx.record("moe.topk_idx", idx)
+        h = ctx.scratch("moe.h", (M, self.di), self.dtype)
+        at = None
+        if self.dtype == torch.bfloat16 and M <= linear.SKINNY_MAX_PAIRS and self.d % 8 == 0 and self.di % 8 == 0:
+            pairs = idx.view(-1)
+            if gemm_skinny(x1, self.weights["wgu"], h, groups=self.E, out_kind=2, max_group_rows=nt, row_group=pairs,
+                           x_div=self.k, glu=self.glu) and \
+                    gemm_skinny(h, self.weights["wd"], y, groups=self.E, max_group_rows=nt, row_group=pairs):
+                at = _term_rows(nt, self.k, bool(self.shared), x1.device)
+        if at is None:
+            offsets = ctx.scratch("moe.offsets", (self.E + 1,), torch.int32)
+            sorted_token = ctx.scratch("moe.sorted_token", (M,), torch.int32)
+            at = ctx.scratch("moe.term_row", (nt * self.terms,), torch.int32)
+            lib.call("tb_moe_dispatch_shared" if self.shared else "tb_moe_dispatch", lib.ptr(idx), lib.ptr(offsets),
+                     lib.ptr(sorted_token), lib.ptr(at), M, self.k, self.E)
+            grouped_matmul(x1, self.weights["wgu"], h, a_rows=sorted_token, group_offsets=offsets, groups=self.E,
+                           swiglu=True, max_group_rows=nt, scratch=ctx.scratch, glu=self.glu)
+            grouped_matmul(h, self.weights["wd"], y, group_offsets=offsets, groups=self.E, max_group_rows=nt)
+        if self.shared:
+            self._shared(ctx, x1, rows[M:])
+        return WeightedRows(rows, at, w, self.terms)
+
     def forward(self, ctx, x1, out, tail=None) -> None:
+        if self.table or self.shared:
+            return self._forward_terms(ctx, x1, tail)
         nt = x1.shape[0]
         M = nt * self.k
         sfx = lib.suffix(self.dtype)
@@ -292,6 +386,22 @@ def _identity_rows(n: int, device) -> torch.Tensor:
     if key not in _IDENTITY_ROWS:
         _IDENTITY_ROWS[key] = torch.arange(n, dtype=torch.int32, device=device)
     return _IDENTITY_ROWS[key]
+
+
+_TERM_ROWS = {}
+
+
+def _term_rows(nt: int, k: int, shared: bool, device) -> torch.Tensor:
+    """The rows of every token's terms where pair (t, j) lies in row t k + j and a shared expert's results in the rows
+    behind, made once per size."""
+    if not shared:
+        return _identity_rows(nt * k, device)
+    key = (nt, k, str(device))
+    if key not in _TERM_ROWS:
+        pairs = torch.arange(nt * k, dtype=torch.int32).view(nt, k)
+        own = nt * k + torch.arange(nt, dtype=torch.int32)
+        _TERM_ROWS[key] = torch.cat([pairs, own[:, None]], dim=1).reshape(-1).contiguous().to(device)
+    return _TERM_ROWS[key]
 
 
 _ONES = {}

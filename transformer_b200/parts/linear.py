@@ -16,9 +16,17 @@ import torch
 from ..csrc import lib
 
 
+GELU_TANH = "gelu_tanh"     # as ``glu``: the tanh form of gelu on the gate, times up
+
+
+def _glu_args(glu):
+    """(alpha, limit, kind) of the launchers for another form of the (gate, up) pair than silu(gate) * up."""
+    return (0.0, 0.0, 3) if glu == GELU_TANH else (float(glu[0]), float(glu[1]), 1)
+
+
 def gemm_simt(a, w, out, *, a_rows=None, group_offsets=None, groups=1, rows=None, out_kind=0, glu=None) -> None:
     """out[m] = a[a_rows[m] or m] . w[g(m)]^T ; w is [N, K] or [G, N(or 2N), K].  ``glu`` = (alpha, limit): the
-    clamped form of the (gate, up) pair instead of swiglu (with out_kind 2)."""
+    clamped form of the (gate, up) pair instead of swiglu, GELU_TANH: gelu(gate) * up (with out_kind 2)."""
     M = out.shape[0] if rows is None else rows
     K = a.shape[-1]
     N = out.shape[-1]
@@ -31,8 +39,7 @@ def gemm_simt(a, w, out, *, a_rows=None, group_offsets=None, groups=1, rows=None
     assert a.stride(-1) == 1 and w.stride(-1) == 1 and out.stride(-1) == 1
     if glu is not None and out_kind == 2:
         lib.call("tb_gemm_simt_glu_" + lib.suffix(a.dtype), lib.ptr(a), lib.ptr(a_rows), lib.ptr(w), lib.ptr(out),
-                 lib.ptr(group_offsets), stride, a.stride(0), ldb, out.stride(0), M, N, K, groups, float(glu[0]),
-                 float(glu[1]))
+                 lib.ptr(group_offsets), stride, a.stride(0), ldb, out.stride(0), M, N, K, groups, *_glu_args(glu))
         return
     lib.call("tb_gemm_simt_" + lib.suffix(a.dtype), lib.ptr(a), lib.ptr(a_rows), lib.ptr(w), lib.ptr(out),
              lib.ptr(group_offsets), stride, a.stride(0), ldb, out.stride(0), M, N, K, groups, out_kind)
@@ -80,8 +87,7 @@ def gemm_skinny(a, w, out, *, a_rows=None, group_offsets=None, groups=1, out_kin
     if glu is not None and out_kind == 2:
         return lib.try_call("tb_gemm_skinny_glu_bf16", lib.ptr(a), lib.ptr(a_rows), lib.ptr(w), lib.ptr(out),
                             lib.ptr(group_offsets), stride, a.stride(0), ldw, out.stride(0), M, N, K, groups,
-                            max_group_rows, lib.ptr(row_group), x_div, 1 if w_is_weight else 0, float(glu[0]),
-                            float(glu[1]))
+                            max_group_rows, lib.ptr(row_group), x_div, 1 if w_is_weight else 0, *_glu_args(glu))
     return lib.try_call("tb_gemm_skinny_bf16", lib.ptr(a), lib.ptr(a_rows), lib.ptr(w), lib.ptr(out),
                         lib.ptr(group_offsets), stride, a.stride(0), ldw, out.stride(0), M, N, K, groups, out_kind,
                         max_group_rows, lib.ptr(row_group), x_div, 1 if w_is_weight else 0)
@@ -95,7 +101,7 @@ def gemm_tc(a, w, out, *, group_offsets=None, groups=1, out_kind=0, glu=None) ->
     assert a.stride(-1) == 1 and w.stride(-1) == 1 and out.stride(-1) == 1 and w.is_contiguous()
     if glu is not None and out_kind == 2:
         return lib.try_call("tb_gemm_tc_glu_bf16", lib.ptr(a), lib.ptr(w), lib.ptr(out), lib.ptr(group_offsets),
-                            a.stride(0), ldw, out.stride(0), M, N, K, groups, float(glu[0]), float(glu[1]))
+                            a.stride(0), ldw, out.stride(0), M, N, K, groups, *_glu_args(glu))
     return lib.try_call("tb_gemm_tc_bf16", lib.ptr(a), lib.ptr(w), lib.ptr(out), lib.ptr(group_offsets),
                         a.stride(0), ldw, out.stride(0), M, N, K, groups, out_kind)
 
@@ -125,7 +131,7 @@ def matmul_nt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w_is_weigh
 def grouped_matmul(a, w, out, *, a_rows=None, group_offsets=None, groups=1, swiglu=False, max_group_rows=0,
                    scratch=None, w_is_weight: bool = True, glu=None) -> None:
     """out[m] = a[a_rows[m] or m] . w[g(m)]^T over rows sorted by group; with swiglu, w[g] holds gate rows
-    then up rows and out = silu(gate) * up (or, with ``glu`` = (alpha, limit), the clamped form of the pair).  max_group_rows: a bound on the rows of one group, if known;
+    then up rows and out = silu(gate) * up (or another form of the pair by ``glu``).  max_group_rows: a bound on the rows of one group, if known;
     scratch(name, shape, dtype): where the prompt kernel may put the gathered rows."""
     kind = 2 if swiglu else 0
     if a.dtype == torch.bfloat16 and out.shape[0] <= SKINNY_MAX_PAIRS and \

@@ -90,15 +90,18 @@ class RMSNorm(Norm):
 
 @NORMS.register("layernorm")
 class LayerNorm(Norm):
-    """params: width, eps, bias (default True), scale (default False).  y = (v - mean v) / sqrt(var v + eps) * weight
+    """params: width, eps, bias (default True), scale (default False), stream (default 1).  y = (v - mean v) / sqrt(var v + eps) * weight
     + bias, the variance being the mean of the squared deviations.  With ``scale`` the result is multiplied channel
     by channel by a further learned vector ("scale": a block's layer scale), which is folded into the bound weight
     and bias (float, once).  Statistics and the residual sum are float; one rounding at the store.  A pending
-    :class:`NormedDelta` of either kind is normed, added and normed again in the same kernel."""
+    :class:`NormedDelta` of either kind is normed, added and normed again in the same kernel.
+
+    :meth:`renew` is the form of a block that norms the stream itself: x <- y = N(stream * x + delta)."""
     graph_safe = True
     launches_only = True
     takes_weighted_rows = True
     takes_normed_delta = True
+    renew_tails = ("terms",)
 
     def __init__(self, params, dtype, device):
         super().__init__(params, dtype, device)
@@ -106,6 +109,7 @@ class LayerNorm(Norm):
         self.eps = float(params["eps"])
         self.bias = bool(params.get("bias", True))
         self.scale = bool(params.get("scale", False))
+        self.stream = float(params.get("stream", 1.0))
 
     def parameters(self):
         decl = {"weight": ParamDecl((self.width,), "norm", "ones")}
@@ -133,6 +137,20 @@ class LayerNorm(Norm):
             post, delta = delta, delta.delta
         post_add_layernorm(self.dtype, x, delta, post, rows, self.weights["weight"], self.weights.get("bias"), self.eps,
                            True, y)
+
+    def renew(self, ctx, x, delta, y, tail=None) -> None:
+        """x <- N(stream * x + delta) in float, y the same rounded to the activation type; ``delta`` a tensor or a
+        :class:`WeightedRows`.  ``tail``: a "terms" :class:`NormTail` of the rows y, computed along the way."""
+        wy = idx = wts = None
+        k = 0
+        if isinstance(delta, WeightedRows):
+            wy, idx, wts, k, delta = delta.rows, delta.index, delta.weights, delta.k, None
+        t = tail
+        pick = (0, 0, 0, 0, 0, 0) if t is None else (lib.ptr(ctx.tok_ids), lib.ptr(t.table), lib.ptr(t.gate),
+                                                     lib.ptr(t.index), lib.ptr(t.scores), t.k)
+        lib.call("tb_renew_layernorm_" + lib.suffix(self.dtype), lib.ptr(x), lib.ptr(delta), lib.ptr(wy), lib.ptr(idx),
+                 lib.ptr(wts), k, self.stream, lib.ptr(self.weights["weight"]), lib.ptr(self.weights.get("bias")), self.eps,
+                 lib.ptr(y), y.shape[0], self.width, *pick)
 
 
 @NORMS.register("none")

@@ -75,3 +75,15 @@ def normal_values(seed: int, name: str, first: int, count: int, std: float) -> n
                     total += ((h >> np.uint64(16 * f)) & np.uint64(0xFFFF)).astype(np.int64)
             out[lo:lo + n] = (total - 4 * 65535).astype(np.float32) * scale
     return out
+
+
+def distinct_rows(seed: int, name: str, rows: int, cols: int, n: int) -> np.ndarray:
+    """int32 [rows, cols] of integers below ``n``, those of a row differing: row i starts at h_i mod n, h_i the i-th
+    counter value of the tensor's stream, and counts on from there."""
+    if cols > n:
+        raise ValueError(f"a row of {cols} different integers needs at least as many, got {n}")
+    base = np.uint64(stream_base(seed, name))
+    with np.errstate(over="ignore"):
+        h = _mix64(base + np.arange(rows, dtype=np.uint64) * np.uint64(G))
+    first = (h % np.uint64(n)).astype(np.int64)
+    return ((first[:, None] + np.arange(cols)[None, :]) % n).astype(np.int32)

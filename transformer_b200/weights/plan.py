@@ -50,7 +50,8 @@ class TensorRule:
     shape: Tuple[int, ...]
     role: str                               # "matrix" | "norm" | "table"
     sources: Tuple[Source, ...]
-    init: str = "normal"                    # how the random-weights mode fills it: "normal" | "ones"
+    init: str = "normal"                    # how the random-weights mode fills it: "normal" | "ones" | "distinct:n"
+                                            # (integers 0 .. n-1, those of a row differing)
     shared_with: Optional[Dest] = None      # when no source is present, reuse this parameter (tied head)
     unused: bool = False                    # a tensor that a file may carry and no part reads: taken note of when it
                                             # is there (so that it is not reported as unexpected), never asked for

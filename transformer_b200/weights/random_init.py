@@ -31,6 +31,8 @@ def _host_piece(name: str, shape, init: str, seed: int, std: float) -> torch.Ten
         for s in shape:
             n *= int(s)
         return torch.from_numpy(counter_random.normal_values(seed, name, 0, n, std)).reshape(tuple(shape))
+    if init.startswith("distinct:"):
+        return torch.from_numpy(counter_random.distinct_rows(seed, name, int(shape[0]), int(shape[1]), int(init[9:])))
     raise ValueError(f"unknown init {init!r}")
 
 
@@ -71,6 +73,9 @@ def random_device_weights(rules: Sequence[TensorRule], seed: int, compute_dtype:
             dtype = storage_dtype(rule.role, compute_dtype)
             if rule.init == "ones":
                 out[rule.dest] = torch.ones(rule.shape, dtype=dtype, device=device)
+                continue
+            if rule.init.startswith("distinct:"):      # a table of integers: small, made on the host
+                out[rule.dest] = _host_piece(rule.canonical.names[0], rule.shape, rule.init, int(seed), std).to(device)
                 continue
             if rule.init != "normal":
                 raise ValueError(f"unknown init {rule.init!r}")
