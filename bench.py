@@ -5,6 +5,7 @@
     python bench.py --design salepel [--sizes s,m]      another design beside Llama-MoE at equal sizes (see bench_design)
     python bench.py --design zufadra [--sizes s,m]      the Zufadra design beside a dense Llama at equal sizes
     python bench.py --design fugavik [--sizes s,m]      the Fugavik design beside Zufadra, Dumalix and Llama-MoE
+    python bench.py --design fofapel [--sizes s,m]      the Fofapel design beside Fugavik, Zufadra and Llama-MoE
 
 The default run has the layer sizes of the LLaMA-MoE-3.5B (4/16) shape (32 layers, width 4096,
 32/32 heads of 128, 16 experts top-4 of width 688, vocabulary 32000, context 4096) with random
@@ -253,6 +254,28 @@ def fugavik_shapes(size):
     return fugavik, zufadra_shapes(size)[0], dumalix_shapes(size)[0], design_shapes(size)[1]
 
 
+def fofapel_shapes(size):
+    """(Fofapel config, Fugavik config, Zufadra config, Llama-MoE config) for a named size.  Every Fofapel layer has both
+    mixers; the feed-forwards alternate between the dense pair and the experts with the shared one.  Fugavik (layer norm
+    fused with the residual sum, the per-head kernel before the windowed attention with a sink, dense and experts'
+    feed-forwards) is the closest model for everything but the recurrence; Zufadra (and Fugavik) has the delta rule, a
+    recurrence with a state of the same size; Llama-MoE the experts of the same sizes."""
+    d, L, H, G, dim, window, rank, ff, E, top, eff, shared = {
+        "s": (1024, 8, 8, 2, 128, 1024, 64, 2816, 8, 2, 512, 512),
+        "m": (2048, 8, 16, 4, 128, 2048, 128, 5632, 16, 4, 704, 1408),
+    }[size]
+    mixer = {"left": {"heads": H, "kv_heads": G, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+                      "rot": {"base": 500000.0, "dims": dim}},
+             "right": {"heads": H, "dim": dim, "decay_rank": rank}, "left_scale": 1.0, "right_scale": 1.0}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "router": {"experts": E, "top": top},
+           "shared": {"ff": shared, "limit": 7.0}}
+    fofapel = {"architecture": "Fofapel", "vocab": 32000, "width": d, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+               "max_context": 8192,
+               "layers": [{"type": "parallel", "mixer": mixer, "mlp": dense if i % 2 == 0 else moe} for i in range(L)]}
+    return fofapel, fugavik_shapes(size)[0], zufadra_shapes(size)[0], design_shapes(size)[1]
+
+
 def bench_design(args):
     """Prefill and decode throughput of another design beside the closest existing model of equal sizes, and the
     device time of every kernel family in one eager step of each (CUDA events around each launch).  One JSON line."""
@@ -267,7 +290,8 @@ def bench_design(args):
     names, shapes = {"salepel": (("salepel", "llama_moe"), design_shapes),
                      "zufadra": (("zufadra", "llama_dense"), zufadra_shapes),
                      "dumalix": (("dumalix", "zufadra_attention", "salepel"), dumalix_shapes),
-                     "fugavik": (("fugavik", "zufadra", "dumalix", "llama_moe"), fugavik_shapes)}[args.design]
+                     "fugavik": (("fugavik", "zufadra", "dumalix", "llama_moe"), fugavik_shapes),
+                     "fofapel": (("fofapel", "fugavik", "zufadra", "llama_moe"), fofapel_shapes)}[args.design]
     out = {"metric": f"prefill and decode tok/s, {names[0]} beside {' and '.join(names[1:])} at equal sizes", "unit": "tokens/s",
            "dtype": "bf16" if args.dtype == "bfloat16" else "fp32", "data": "synthetic: random weights, random token ids",
            "peaks": pk, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx0, "steps": K, "warmup": W,
@@ -363,7 +387,7 @@ def main():
                     help="layer sizes: the benchmark's (default) or another shape BASELINE.json names")
     ap.add_argument("--prompt-max", type=int, default=0, help="longest prompt drawn (default: the shape's own)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS)
-    ap.add_argument("--design", default=None, choices=["salepel", "zufadra", "dumalix", "fugavik"],
+    ap.add_argument("--design", default=None, choices=["salepel", "zufadra", "dumalix", "fugavik", "fofapel"],
                     help="instead of the default workload: this design beside the closest existing model at equal "
                          "sizes (prefill of --prefill-tokens, decode at --batch; sizes from --sizes)")
     ap.add_argument("--sizes", default="s,m", help="with --design: which of the named sizes (s, m)")

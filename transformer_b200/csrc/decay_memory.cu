@@ -11,6 +11,7 @@
 // State of one slot (floats): S [H][dim][dim], then the last input [width]; the pitch is a multiple of four.
 //
 //   shift_mix_kernel    all mixes of a token at once, and the group lists of the product that follows (a matrix per mix)
+//   decay_tanh_kernel   prompts: tanh(a) for the product with W2
 //   decay_prep_kernel   prompts: decays and bonuses; one float record per (token, head) for the scan, r | k | w | bonus
 //   decay_scan_kernel   prompts: the recurrence token by token, a block = a sequence x a head x some columns of S, whose
 //                       rows are split over adjacent lanes, in registers; the lanes' sums meet only in the output, so
@@ -22,9 +23,9 @@
 #include "attention_prefill.cuh"        // cp_async16, cp_async_commit, cp_async_wait
 
 constexpr int DM_MIXES = 5;             // r, k, v, gate, decay
-constexpr int DM_TOK = 4;               // tokens the scan stages per barrier
+constexpr int DM_TOK = 8;               // tokens of a stage of the scan
+constexpr int DM_STAGES = 4;            // stages in flight or in use
 constexpr int DM_SCAN = 128;            // threads of a scan block
-constexpr int DM_PREP_TOK = 8;          // tokens of a prep block
 
 __host__ __device__ inline int dm_rows(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 __host__ __device__ inline int dm_record(int dim) { return 3 * dm_rows(dim) + 4; }
@@ -111,6 +112,26 @@ static int shift_mix_launch(const void* x, const float* mu, const float* state, 
     return tb_last_error();
 }
 
+template <typename T, int V>
+__device__ __forceinline__ void dm_load(const T* p, float (&f)[V]) {
+    if constexpr (V == 1) {
+        f[0] = ldf(p);
+    } else if constexpr (sizeof(T) == 2) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+    } else {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    }
+}
+template <int V>
+__device__ __forceinline__ void dm_store(float* p, const float (&f)[V]) {
+    if constexpr (V == 1) *p = f[0];
+    else *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+
 // ---- decays ------------------------------------------------------------------------------------------------
 // w0 + W2 row . ta for DT tokens at once; ta [DT][rank] in shared memory
 template <typename T, int DT>
@@ -139,81 +160,87 @@ __device__ __forceinline__ void decay_dot(const T* __restrict__ w2row, const flo
     }
 }
 
+// tanh of the decay's first projection, ready for the product with W2: in the activations' type a value is stored as the
+// sum of two (what its rounding leaves goes into the second half of the row, and the product's weight holds W2 twice), so
+// the product loses nothing that matters; in float it is stored as it is.
+template <typename T>
+__global__ void __launch_bounds__(256) decay_tanh_kernel(const float* __restrict__ a, int lda, T* __restrict__ out, int nt,
+                                                         int rank, int ldo) {
+    pdl_sync();
+    const int n = nt * ldo;
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+        const int t = i / ldo, q = i - t * ldo;
+        const int half = sizeof(T) == 2 ? ldo / 2 : ldo;        // entries of a half, beyond rank zero
+        const int e = q < half ? q : q - half;
+        float v = 0.f;
+        if (e < rank) {
+            v = tanhf(a[(size_t)t * lda + e]);
+            if (q >= half) {
+                T hi;
+                stf(&hi, v);
+                v -= ldf(&hi);
+            }
+        }
+        stf(out + i, v);
+    }
+}
+
 struct DecayArgs {
     const void* z;          // [4 nt, H dim]: r, k, v, gate, nt rows each
-    const float* a;         // [nt, lda] the decay's first projection
-    const void* w2;         // [H dim, rank]
+    const float* pre;       // [nt, H dim]  W2 tanh(.)
     const float* w0;        // [H dim]
     const float* u;         // [H dim]
     float* rec;             // [nt, H, dm_record]
     float* vals;            // [nt, H, dm_vpitch]
-    int nt, lda, H, dim, rank;
+    int nt, H, dim;
 };
 
-// A block = DM_PREP_TOK consecutive tokens x one head; a thread takes a key channel (or every 256th).
-template <typename T>
+// A warp per (token, head): the record and the values; four neighbouring entries a lane and access where the layout
+// allows it (VEC).
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) decay_prep_kernel(const DecayArgs p) {
     pdl_sync();
-    extern __shared__ __align__(16) float dm_sm[];        // [DM_PREP_TOK][rank] tanh(a)
-    __shared__ float part[8][DM_PREP_TOK];
-    const int t0 = blockIdx.x * DM_PREP_TOK, h = blockIdx.y;
-    const int n = min(DM_PREP_TOK, p.nt - t0), dim = p.dim, hd = p.H * dim;
-    const int DP = dm_rows(dim), PER = dm_record(dim), VP = dm_vpitch(dim);
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    for (int i = threadIdx.x; i < DM_PREP_TOK * p.rank; i += blockDim.x) {
-        const int tt = i / p.rank, q = i - tt * p.rank;
-        dm_sm[i] = tt < n ? tanhf(p.a[(size_t)(t0 + tt) * p.lda + q]) : 0.f;
-    }
-    __syncthreads();
-    const T* z = static_cast<const T*>(p.z);
-    float bonus[DM_PREP_TOK];
+    constexpr int V = VEC ? 4 : 1;
+    const int lane = threadIdx.x & 31;
+    const int row = blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (row >= p.nt * p.H) return;
+    const int t = row / p.H, h = row - t * p.H, dim = p.dim, hd = p.H * dim;
+    const int DP = dm_rows(dim), VP = dm_vpitch(dim);
+    float* rec = p.rec + (size_t)row * dm_record(dim);
+    float* vals = p.vals + (size_t)row * VP;
+    const T* z = static_cast<const T*>(p.z) + (size_t)t * hd + h * dim;
+    const size_t part = (size_t)p.nt * hd;
+    float bonus = 0.f;
+    for (int c = lane * V; c < max(DP, VP); c += 32 * V) {
+        float r[V], k[V], v[V], w[V];
 #pragma unroll
-    for (int tt = 0; tt < DM_PREP_TOK; ++tt) bonus[tt] = 0.f;
-    for (int c = threadIdx.x; c < DP; c += blockDim.x) {
-        const bool live = c < dim;
-        const int hc = h * dim + c;
-        float acc[DM_PREP_TOK];
-        float uc = 0.f;
-        if (live) {
-            decay_dot<T, DM_PREP_TOK>(static_cast<const T*>(p.w2) + (size_t)hc * p.rank, dm_sm, p.rank, p.w0[hc], acc);
-            uc = p.u[hc];
+        for (int e = 0; e < V; ++e) {
+            r[e] = k[e] = v[e] = 0.f;
+            w[e] = 1.f;
         }
+        if (c < dim) {
+            float pre[V], w0[V], u[V];
+            dm_load<T, V>(z + c, r);
+            dm_load<T, V>(z + part + c, k);
+            dm_load<T, V>(z + 2 * part + c, v);
+            dm_load<float, V>(p.pre + (size_t)t * hd + h * dim + c, pre);
+            dm_load<float, V>(p.w0 + h * dim + c, w0);
+            dm_load<float, V>(p.u + h * dim + c, u);
 #pragma unroll
-        for (int tt = 0; tt < DM_PREP_TOK; ++tt) {
-            if (tt >= n) break;
-            const int t = t0 + tt;
-            float* r = p.rec + ((size_t)t * p.H + h) * PER;
-            float rv = 0.f, kv = 0.f, w = 1.f, vv = 0.f;
-            if (live) {
-                rv = ldf(z + (size_t)t * hd + hc);
-                kv = ldf(z + ((size_t)p.nt + t) * hd + hc);
-                vv = ldf(z + ((size_t)2 * p.nt + t) * hd + hc);
-                w = expf(-expf(acc[tt]));
-                bonus[tt] += rv * uc * kv;
+            for (int e = 0; e < V; ++e) {
+                w[e] = expf(-expf(pre[e] + w0[e]));
+                bonus += r[e] * u[e] * k[e];
             }
-            r[c] = rv;
-            r[DP + c] = kv;
-            r[2 * DP + c] = w;
-            if (c < VP) p.vals[((size_t)t * p.H + h) * VP + c] = vv;
         }
+        if (c < DP) {
+            dm_store<V>(rec + c, r);
+            dm_store<V>(rec + DP + c, k);
+            dm_store<V>(rec + 2 * DP + c, w);
+        }
+        if (c < VP) dm_store<V>(vals + c, v);
     }
-    // VP may exceed DP only for dim <= 16
-    if (VP > DP)
-        for (int i = threadIdx.x; i < n * (VP - DP); i += blockDim.x)
-            p.vals[((size_t)(t0 + i / (VP - DP)) * p.H + h) * VP + DP + i % (VP - DP)] = 0.f;
-#pragma unroll
-    for (int tt = 0; tt < DM_PREP_TOK; ++tt) {
-        const float s = warp_sum(bonus[tt]);
-        if (lane == 0) part[warp][tt] = s;
-    }
-    __syncthreads();
-    for (int i = threadIdx.x; i < n * 4; i += blockDim.x) {
-        const int tt = i >> 2, j = i & 3;
-        float s = 0.f;
-        if (j == 0)
-            for (int w = 0; w < warps; ++w) s += part[w][tt];
-        p.rec[((size_t)(t0 + tt) * p.H + h) * PER + 3 * DP + j] = s;
-    }
+    bonus = warp_sum(bonus);
+    if (lane < 4) rec[3 * DP + lane] = lane == 0 ? bonus : 0.f;
 }
 
 // ---- the scan ------------------------------------------------------------------------------------------------
@@ -229,89 +256,144 @@ struct DecayScanArgs {
     int H, dim, width;
 };
 
-// RPT rows of a column per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)), DM_SCAN / SPLIT columns a block.
-template <typename T, int RPT, int SPLIT>
+// two floats in one register pair, and the hardware's packed multiply-add on them
+union F2 {
+    float2 f;
+    unsigned long long u;
+};
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+    F2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d.u) : "l"(a.u), "l"(b.u), "l"(c.u));
+    return d;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+    F2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d.u) : "l"(a.u), "l"(b.u));
+    return d;
+}
+
+// RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): DM_SCAN / SPLIT * C columns a
+// block.  The records of DM_TOK tokens at a time are copied to shared memory by cp.async, DM_STAGES - 1 stages ahead.  A
+// token needs no reduction: every lane keeps its rows' share of the outputs of a whole stage, and the DM_TOK * C shares
+// are then summed over the column's lanes so that each lane ends with some of the sums (fewer shuffles than sums).
+template <typename T, int RPT, int SPLIT, int C>
 __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs a) {
     pdl_sync();
     constexpr int DP = RPT * SPLIT;
-    constexpr int COLS = DM_SCAN / SPLIT;
+    constexpr int COLS = DM_SCAN / SPLIT * C;
     constexpr int PER = 3 * DP + 4;
     constexpr int ROW = PER + COLS;
     constexpr int ROW4 = ROW / 4;
-    __shared__ __align__(16) float sm[2][DM_TOK][ROW];
+    constexpr int NV = DM_TOK * C;
+    static_assert(NV % SPLIT == 0 && COLS % 4 == 0, "every lane ends with as many sums");
+    extern __shared__ __align__(16) float dm_sm[];      // [DM_STAGES][DM_TOK][ROW]
     const int b = blockIdx.x, h = blockIdx.y;
-    const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT;
+    const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT * C;
     const int col0 = blockIdx.z * COLS, col = col0 + cl;
     const int dim = a.dim, H = a.H;
-    const bool has_col = col < dim;
     const int t0 = a.seq_start[b], t1 = a.seq_start[b + 1];
     if (t0 >= t1) return;
     const int VP = dm_vpitch(dim);
     float* slot = a.state + (size_t)a.slots[b] * a.pitch;
     float* S = slot + (size_t)h * dim * dim;
-    float s[RPT];
+    F2 s[C][RPT / 2];                                   // rows 2i, 2i + 1 of this lane's
 #pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-        const int r = ((i >> 2) * SPLIT + part) * 4 + (i & 3);
-        s[i] = (r < dim && has_col) ? S[(size_t)r * dim + col] : 0.f;
-    }
-    auto issue = [&](int ts, int par) {
-        const int ntok = min(DM_TOK, t1 - ts);
-        for (int idx = tid; idx < ntok * ROW4; idx += DM_SCAN) {
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int i = 0; i < RPT / 2; ++i) {
+            const int r = ((i >> 1) * SPLIT + part) * 4 + (i & 1) * 2;
+            s[c][i].f.x = (r < dim && col + c < dim) ? S[(size_t)r * dim + col + c] : 0.f;
+            s[c][i].f.y = (r + 1 < dim && col + c < dim) ? S[(size_t)(r + 1) * dim + col + c] : 0.f;
+        }
+    auto issue = [&](int ts) {
+        const int n = min(DM_TOK, t1 - ts);
+        float* to = dm_sm + (size_t)((ts - t0) / DM_TOK % DM_STAGES) * (DM_TOK * ROW);
+        for (int idx = tid; idx < n * ROW4; idx += DM_SCAN) {
             const int tt = idx / ROW4, e4 = idx - tt * ROW4;
             // columns behind the padded row of values are left alone: no column of the head reads them
             if (e4 >= PER / 4 && col0 + (e4 - PER / 4) * 4 >= VP) continue;
             const float* src = e4 < PER / 4 ? a.rec + ((size_t)(ts + tt) * H + h) * PER + e4 * 4
                                             : a.vals + ((size_t)(ts + tt) * H + h) * VP + col0 + (e4 - PER / 4) * 4;
-            cp_async16((uint32_t)__cvta_generic_to_shared(&sm[par][tt][e4 * 4]), src);
+            cp_async16((uint32_t)__cvta_generic_to_shared(to + tt * ROW + e4 * 4), src);
         }
-        cp_async_commit();
+        // tokens behind the last: nothing is written, nothing fades, nothing is read (so that a stage has no branches)
+        for (int idx = n * ROW + tid; idx < DM_TOK * ROW; idx += DM_SCAN) {
+            const int e = idx % ROW;
+            to[idx] = e >= 2 * DP && e < 3 * DP ? 1.f : 0.f;
+        }
     };
-    issue(t0, 0);
-    for (int ts = t0, st = 0; ts < t1; ts += DM_TOK, ++st) {
-        const int par = st & 1;
-        cp_async_wait<0>();
+#pragma unroll
+    for (int q = 0; q < DM_STAGES - 1; ++q) {
+        if (t0 + q * DM_TOK < t1) issue(t0 + q * DM_TOK);
+        cp_async_commit();
+    }
+    for (int ts = t0; ts < t1; ts += DM_TOK) {
+        cp_async_wait<DM_STAGES - 2>();
         __syncthreads();            // this stage has landed for everyone, and everyone is done with the stage before
-        if (ts + DM_TOK < t1) issue(ts + DM_TOK, par ^ 1);
-        const int ntok = min(DM_TOK, t1 - ts);
-        float o[DM_TOK];
+        if (ts + (DM_STAGES - 1) * DM_TOK < t1) issue(ts + (DM_STAGES - 1) * DM_TOK);
+        cp_async_commit();
+        const float* stage = dm_sm + (size_t)((ts - t0) / DM_TOK % DM_STAGES) * (DM_TOK * ROW);
+        const int n = min(DM_TOK, t1 - ts);
+        float o[NV];
 #pragma unroll
         for (int tt = 0; tt < DM_TOK; ++tt) {
-            o[tt] = 0.f;
-            if (tt >= ntok) continue;
-            const float* row = &sm[par][tt][0];
-            const float4* R4 = reinterpret_cast<const float4*>(row);
-            const float4* K4 = reinterpret_cast<const float4*>(row + DP);
-            const float4* W4 = reinterpret_cast<const float4*>(row + 2 * DP);
-            const float v = row[PER + cl];
-            float d4[4] = {0.f, 0.f, 0.f, 0.f};
+            const float* row = stage + tt * ROW;
+            F2 v[C], d[C];
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+                v[c].f.x = v[c].f.y = row[PER + cl + c];
+                d[c].f.x = d[c].f.y = 0.f;
+            }
 #pragma unroll
             for (int i4 = 0; i4 < RPT / 4; ++i4) {
                 const int ch = i4 * SPLIT + part;
-                const float4 r = R4[ch], k = K4[ch], w = W4[ch];
-                float* si = s + i4 * 4;
-                d4[0] += si[0] * r.x; d4[1] += si[1] * r.y; d4[2] += si[2] * r.z; d4[3] += si[3] * r.w;
-                si[0] = si[0] * w.x + k.x * v; si[1] = si[1] * w.y + k.y * v;
-                si[2] = si[2] * w.z + k.z * v; si[3] = si[3] * w.w + k.w * v;
+                union { float4 f; F2 p[2]; } r, k, w;
+                r.f = reinterpret_cast<const float4*>(row)[ch];
+                k.f = reinterpret_cast<const float4*>(row + DP)[ch];
+                w.f = reinterpret_cast<const float4*>(row + 2 * DP)[ch];
+#pragma unroll
+                for (int c = 0; c < C; ++c)
+#pragma unroll
+                    for (int q = 0; q < 2; ++q) {
+                        F2& si = s[c][i4 * 2 + q];
+                        d[c] = fma2(si, r.p[q], d[c]);
+                        si = fma2(si, w.p[q], mul2(k.p[q], v[c]));
+                    }
             }
-            o[tt] = (d4[0] + d4[1]) + (d4[2] + d4[3]);
+#pragma unroll
+            for (int c = 0; c < C; ++c) o[tt * C + c] = d[c].f.x + d[c].f.y;
+        }
+        // sum over the column's lanes: at every step a lane hands half of its values over and keeps the other half
+#pragma unroll
+        for (int step = SPLIT / 2, left = NV; step > 0; step >>= 1) {
+            left >>= 1;
+            const bool upper = (part & step) != 0;
+#pragma unroll
+            for (int j = 0; j < NV / 2; ++j) {
+                if (j >= left) break;
+                const float give = upper ? o[j] : o[j + left], keep = upper ? o[j + left] : o[j];
+                o[j] = keep + __shfl_xor_sync(0xffffffffu, give, step);
+            }
         }
 #pragma unroll
-        for (int tt = 0; tt < DM_TOK; ++tt)
-#pragma unroll
-            for (int q = 1; q < SPLIT; q <<= 1) o[tt] += __shfl_xor_sync(0xffffffffu, o[tt], q);
-#pragma unroll
-        for (int tt = 0; tt < DM_TOK; ++tt)
-            if (tt < ntok && part == (tt & (SPLIT - 1)) && has_col) {
-                const float* row = &sm[par][tt][0];
-                a.out[((size_t)(ts + tt) * H + h) * dim + col] = o[tt] + row[3 * DP] * row[PER + cl];
+        for (int j = 0; j < NV / SPLIT; ++j) {
+            const int idx = part * (NV / SPLIT) + j, tt = idx / C, c = idx % C;
+            if (tt < n && col + c < dim) {
+                const float* row = stage + tt * ROW;
+                a.out[((size_t)(ts + tt) * H + h) * dim + col + c] = o[j] + row[3 * DP] * row[PER + cl + c];
             }
+        }
     }
 #pragma unroll
-    for (int i = 0; i < RPT; ++i) {
-        const int r = ((i >> 2) * SPLIT + part) * 4 + (i & 3);
-        if (r < dim && has_col) S[(size_t)r * dim + col] = s[i];
-    }
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int i = 0; i < RPT / 2; ++i) {
+            const int r = ((i >> 1) * SPLIT + part) * 4 + (i & 1) * 2;
+            if (col + c < dim) {
+                if (r < dim) S[(size_t)r * dim + col + c] = s[c][i].f.x;
+                if (r + 1 < dim) S[(size_t)(r + 1) * dim + col + c] = s[c][i].f.y;
+            }
+        }
     if (h == 0 && blockIdx.z == 0) {        // the mixes have read the old one
         const T* last = static_cast<const T*>(a.x) + (size_t)(t1 - 1) * a.width;
         float* to = slot + (size_t)H * dim * dim;
@@ -319,15 +401,22 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
     }
 }
 
-static int dm_lanes_override = 0;       // measurements: lanes per column whatever the batch (0: by the rule below)
-
-template <typename T, int RPT, int SPLIT>
-static void decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
-    dim3 grid(B, a.H, (a.dim + DM_SCAN / SPLIT - 1) / (DM_SCAN / SPLIT));
+template <typename T, int RPT, int SPLIT, int C>
+static int decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
+    constexpr int COLS = DM_SCAN / SPLIT * C;
+    const size_t smem = (size_t)DM_STAGES * DM_TOK * (3 * RPT * SPLIT + 4 + COLS) * sizeof(float);
+    static bool configured = false;
+    if (smem > 48 * 1024 && !configured) {
+        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    dim3 grid(B, a.H, (a.dim + COLS - 1) / COLS);
     if (early)
-        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT>), grid, DM_SCAN, 0, s, a);
+        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT, C>), grid, DM_SCAN, smem, s, a);
     else        // prompts: the blocks run for the whole sequence and want an SM each (see tb_launch_plain)
-        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT>, grid, dim3(DM_SCAN), 0, s, a);
+        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT, C>, grid, dim3(DM_SCAN), smem, s, a);
+    return tb_last_error();
 }
 
 template <typename T>
@@ -335,37 +424,35 @@ static int decay_scan_launch(const DecayScanArgs& a, int nt, int B, cudaStream_t
     if (B < 0 || a.H <= 0 || a.dim <= 0 || a.width <= 0 || a.pitch < dm_state(a.H, a.dim, a.width)) return TB_ERR_ARG;
     if (a.dim > 256) return TB_ERR_UNSUPPORTED;
     if (B == 0) return 0;
-    const int rows = dm_rows(a.dim);
-    int lanes = rows >= 128 ? 16 : rows >= 32 ? 8 : 4;
-    if (dm_lanes_override > 0) lanes = dm_lanes_override;
     const bool early = nt <= 2 * B;
-    if (lanes > rows / 4) lanes = rows / 4;
-    if (rows / lanes > 32) lanes = rows / 32;
-    switch (rows / lanes * 100 + lanes) {       // rows per thread, lanes per column
-        case 4 * 100 + 4: decay_scan_go<T, 4, 4>(a, B, early, s); break;
-        case 8 * 100 + 4: decay_scan_go<T, 8, 4>(a, B, early, s); break;
-        case 4 * 100 + 8: decay_scan_go<T, 4, 8>(a, B, early, s); break;
-        case 16 * 100 + 4: decay_scan_go<T, 16, 4>(a, B, early, s); break;
-        case 8 * 100 + 8: decay_scan_go<T, 8, 8>(a, B, early, s); break;
-        case 4 * 100 + 16: decay_scan_go<T, 4, 16>(a, B, early, s); break;
-        case 32 * 100 + 4: decay_scan_go<T, 32, 4>(a, B, early, s); break;
-        case 16 * 100 + 8: decay_scan_go<T, 16, 8>(a, B, early, s); break;
-        case 8 * 100 + 16: decay_scan_go<T, 8, 16>(a, B, early, s); break;
-        case 32 * 100 + 8: decay_scan_go<T, 32, 8>(a, B, early, s); break;
-        case 16 * 100 + 16: decay_scan_go<T, 16, 16>(a, B, early, s); break;
-        default: return TB_ERR_UNSUPPORTED;
+    switch (dm_rows(a.dim)) {
+        case 16: return decay_scan_go<T, 4, 4, 1>(a, B, early, s);
+        case 32: return decay_scan_go<T, 4, 8, 1>(a, B, early, s);
+        case 64: return decay_scan_go<T, 8, 8, 1>(a, B, early, s);
+        case 128: return decay_scan_go<T, 8, 16, 2>(a, B, early, s);
+        default: return decay_scan_go<T, 16, 16, 2>(a, B, early, s);
     }
-    return tb_last_error();
 }
 
 template <typename T>
 static int decay_prep_launch(const DecayArgs& p, cudaStream_t s) {
-    if (p.nt < 0 || p.H <= 0 || p.dim <= 0 || p.rank <= 0 || p.lda < p.rank) return TB_ERR_ARG;
+    if (p.nt < 0 || p.H <= 0 || p.dim <= 0) return TB_ERR_ARG;
     if (p.dim > 256) return TB_ERR_UNSUPPORTED;
-    const size_t smem = (size_t)DM_PREP_TOK * p.rank * sizeof(float);
-    if (smem > 48 * 1024 || (p.rank % 8 == 0 && ((uintptr_t)p.w2 & 15))) return TB_ERR_UNSUPPORTED;
     if (p.nt == 0) return 0;
-    TB_LAUNCH((decay_prep_kernel<T>), dim3((p.nt + DM_PREP_TOK - 1) / DM_PREP_TOK, p.H), max(32, dm_rows(p.dim)), smem, s, p);
+    const bool vec = p.dim % 4 == 0 &&
+                     (((uintptr_t)p.z | (uintptr_t)p.pre | (uintptr_t)p.w0 | (uintptr_t)p.u) & 15) == 0;
+    const int grid = (int)(((long long)p.nt * p.H + 7) / 8);
+    if (vec) TB_LAUNCH((decay_prep_kernel<T, true>), grid, 256, 0, s, p);
+    else TB_LAUNCH((decay_prep_kernel<T, false>), grid, 256, 0, s, p);
+    return tb_last_error();
+}
+template <typename T>
+static int decay_tanh_launch(const float* a, int lda, void* out, int nt, int rank, int ldo, cudaStream_t s) {
+    if (nt < 0 || rank <= 0 || lda < rank || ldo < rank * (sizeof(T) == 2 ? 2 : 1) || (sizeof(T) == 2 && ldo % 2)) return TB_ERR_ARG;
+    if (nt == 0) return 0;
+    const long long n = (long long)nt * ldo;
+    if (n > (1ll << 30)) return TB_ERR_UNSUPPORTED;
+    TB_LAUNCH((decay_tanh_kernel<T>), (int)((n + 255) / 256 > 1184 ? 1184 : (n + 255) / 256), 256, 0, s, a, lda, (T*)out, nt, rank, ldo);
     return tb_last_error();
 }
 
@@ -509,11 +596,6 @@ extern "C" {
 int tb_decay_state_size(int H, int dim, int width) { return (int)dm_state(H, dim, width); }
 int tb_decay_record_size(int dim) { return dm_record(dim); }
 int tb_decay_value_pitch(int dim) { return dm_vpitch(dim); }
-// For measurements: lanes per column in the scan whatever the batch; 0 gives the choice back to the rule.
-int tb_decay_scan_lanes(int lanes) {
-    dm_lanes_override = lanes;
-    return 0;
-}
 // out [5, nt, d]: the mixes of every token; offsets [groups + 1] and row_group [groups nt] (may be null): the lists by
 // which one grouped product multiplies the first `groups` of them with a matrix each.  `at`: where in a slot's state the
 // last input lies.
@@ -524,10 +606,13 @@ int tb_decay_scan_lanes(int lanes) {
         return shift_mix_launch<T>(x, mu, state, pitch, at, out, offsets, row_group, groups, tok_seq, seq_start,      \
                                    slots, nt, d, s);                                                                  \
     }                                                                                                                 \
-    int tb_decay_prep_##SFX(const void* z, const float* a, int lda, const void* w2, const float* w0, const float* u,  \
-                            float* rec, float* vals, int nt, int H, int dim, int rank, cudaStream_t s) {              \
+    int tb_decay_tanh_##SFX(const float* a, int lda, void* out, int nt, int rank, int ldo, cudaStream_t s) {          \
+        return decay_tanh_launch<T>(a, lda, out, nt, rank, ldo, s);                                                   \
+    }                                                                                                                 \
+    int tb_decay_prep_##SFX(const void* z, const float* pre, const float* w0, const float* u, float* rec,             \
+                            float* vals, int nt, int H, int dim, cudaStream_t s) {                                    \
         if (((uintptr_t)rec | (uintptr_t)vals) & 15) return TB_ERR_ARG;                                               \
-        return decay_prep_launch<T>(DecayArgs{z, a, w2, w0, u, rec, vals, nt, lda, H, dim, rank}, s);                 \
+        return decay_prep_launch<T>(DecayArgs{z, pre, w0, u, rec, vals, nt, H, dim}, s);                              \
     }                                                                                                                 \
     int tb_decay_scan_##SFX(const float* rec, const float* vals, float* state, long long pitch, float* out,           \
                             const void* x, int width, const int* seq_start, const int* slots, int nt, int B, int H,   \
@@ -550,6 +635,8 @@ TB_DECAY(bf16, __nv_bfloat16)
 #include "tape.h"
 TB_TAPE_REGISTER(tb_shift_mix_f32)
 TB_TAPE_REGISTER(tb_shift_mix_bf16)
+TB_TAPE_REGISTER(tb_decay_tanh_f32)
+TB_TAPE_REGISTER(tb_decay_tanh_bf16)
 TB_TAPE_REGISTER(tb_decay_prep_f32)
 TB_TAPE_REGISTER(tb_decay_prep_bf16)
 TB_TAPE_REGISTER(tb_decay_scan_f32)

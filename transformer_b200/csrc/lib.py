@@ -86,7 +86,8 @@ _SIGNATURES: Dict[str, str] = {
     "tb_attention_window_heads_bf16": "pppppppppppiiiiiiiiiiiiffipppifi",
     "tb_attention_window_mma_heads_bf16": "pppppppppppiiiiiiiiiiiiffipppifi",
     "tb_shift_mix_f32": "pppllpppipppii", "tb_shift_mix_bf16": "pppllpppipppii",
-    "tb_decay_prep_f32": "ppipppppiiii", "tb_decay_prep_bf16": "ppipppppiiii",
+    "tb_decay_tanh_f32": "pipiii", "tb_decay_tanh_bf16": "pipiii",
+    "tb_decay_prep_f32": "ppppppiii", "tb_decay_prep_bf16": "ppppppiii",
     "tb_decay_scan_f32": "ppplppippiiii", "tb_decay_scan_bf16": "ppplppippiiii",
     "tb_decay_step_f32": "ppipippppfplpippiiiii", "tb_decay_step_bf16": "ppipippppfplpippiiiii",
     "tb_post_add_layernorm_router_f32": "pppppippfipppfipiippppiii",
@@ -111,7 +112,7 @@ class TapeMap(ctypes.Structure):
     _fields_ = [("base", ctypes.c_ulonglong), ("size", ctypes.c_ulonglong), ("delta", ctypes.c_longlong)]
 
 
-_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i", "tb_decay_value_pitch": "i", "tb_decay_scan_lanes": "i",
+_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i", "tb_decay_value_pitch": "i",
               "tb_attention_window_mma_tile_tokens": "ii", "tb_delta_state_size": "iiiii", "tb_delta_record_size": "i", "tb_delta_scan_lanes": "i", "tb_delta_value_pitch": "i", "tb_mlstm_state_size": "ii", "tb_latent_attention_tile_tokens": "i", "tb_attention_tile_tokens": "ii", "tb_gemm_tc_status": "", "tb_attention_prefill_tile_tokens": "",
               "tb_attention_tc_tile_tokens": ""}
 

@@ -46,6 +46,8 @@ class DecayMemory(Mixer):
         if self.rank > 1024:
             raise ValueError(f"the decaying memory's kernels take ranks up to 1024, got {self.rank}")
         self.rows_width = self.hd = self.H * self.dim
+        # a row of tanh values for the product with W2: in bfloat16 two halves (the value, what its rounding left)
+        self.tanh_width = self.rank if dtype == torch.float32 else 2 * ((self.rank + 3) // 4 * 4)
 
     def parameters(self):
         return {
@@ -61,6 +63,12 @@ class DecayMemory(Mixer):
 
     def bind(self, tensors) -> None:
         super().bind(tensors)
+        w2 = self.weights["w2"]
+        if self.dtype == torch.float32:
+            self.weights["w2_tanh"] = w2
+        else:       # what tanh's rounding leaves is a second half of the product's rows: W2 stands there again
+            half = torch.cat([w2, w2.new_zeros((self.hd, self.tanh_width // 2 - self.rank))], dim=1)
+            self.weights["w2_tanh"] = torch.cat([half, half], dim=1).contiguous()
         if self.out_scale != 1.0:
             self.weights["norm"] = (self.weights["norm"].float() * self.out_scale).contiguous()
 
@@ -92,8 +100,12 @@ class DecayMemory(Mixer):
             return
         rec = ctx.scratch("decay.rec", (nt, H, lib.decay_record_size(self.dim)), torch.float32)
         vals = ctx.scratch("decay.v", (nt, H, lib.decay_value_pitch(self.dim)), torch.float32)
-        lib.call("tb_decay_prep_" + sfx, lib.ptr(z), lib.ptr(a), self.rank, lib.ptr(w["w2"]), lib.ptr(w["w0"]),
-                 lib.ptr(w["u"]), lib.ptr(rec), lib.ptr(vals), nt, H, self.dim, self.rank)
+        th = ctx.scratch("decay.tanh", (nt, self.tanh_width), self.dtype)
+        lib.call("tb_decay_tanh_" + sfx, lib.ptr(a), self.rank, lib.ptr(th), nt, self.rank, self.tanh_width)
+        pre = ctx.scratch("decay.pre", (nt, hd), torch.float32)
+        matmul_nt(th, w["w2_tanh"], pre)                                    # float out
+        lib.call("tb_decay_prep_" + sfx, lib.ptr(z), lib.ptr(pre), lib.ptr(w["w0"]), lib.ptr(w["u"]), lib.ptr(rec),
+                 lib.ptr(vals), nt, H, self.dim)
         o = ctx.scratch("decay.o", (nt, hd), torch.float32)
         lib.call("tb_decay_scan_" + sfx, lib.ptr(rec), lib.ptr(vals), lib.ptr(state), pitch, lib.ptr(o), lib.ptr(x1), d,
                  lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, H, self.dim)
