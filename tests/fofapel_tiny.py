@@ -207,21 +207,29 @@ def as_bfloat16(x):
     return x.bfloat16().to(x.dtype)
 
 
-def check_request(cfg, tensors, tokens, got_rows, dtype, label=""):
-    """got_rows: {position: logits row of the engine}."""
-    ref = FP.forward(cfg, tensors, tokens)
-    diff = {p: float((torch.as_tensor(row).double() - ref[p]).abs().max()) for p, row in sorted(got_rows.items())}
+def check_requests(cfg, tensors, requests, dtype, label=""):
+    """requests: [(tokens, {position: logits row of the engine})], held to the rules together (a request of a few tokens
+    alone says little about what rounding costs the model)."""
+    diffs, lost, top = [], [], 0.0
+    for i, (tokens, got_rows) in enumerate(requests):
+        ref = FP.forward(cfg, tensors, tokens)
+        top = max(top, float(ref.abs().max()))
+        diffs += [(float((torch.as_tensor(row).double() - ref[p]).abs().max()), i, p) for p, row in sorted(got_rows.items())]
+        if dtype != "float32":
+            lost += (FP.forward(cfg, tensors, tokens, store=as_bfloat16) - ref).abs().max(dim=1).values.tolist()
     if dtype == "float32":
-        tol = FP32_TOL * max(1.0, float(ref.abs().max()) / 10.0)
+        tol = FP32_TOL * max(1.0, top / 10.0)
     else:
-        lost = (FP.forward(cfg, tensors, tokens, store=as_bfloat16) - ref).abs().max(dim=1).values
-        tol = BF16_EACH * float(lost.max())
-        mean, rule = sum(diff.values()) / len(diff), BF16_MEAN * float(lost.mean())
-        if len(diff) >= 20:
+        tol, rule = BF16_EACH * max(lost), BF16_MEAN * sum(lost) / len(lost)
+        mean = sum(v for v, _, _ in diffs) / len(diffs)
+        if len(diffs) >= 20:
             assert mean <= rule, f"{label}: mean |diff| {mean:.3e} > {rule:.3e}"
-    for p, v in diff.items():
-        assert v <= tol, f"{label}: position {p} (first wrong of the request): |diff| {v:.3e} > {tol:.3e}"
-    return max(diff.values())
+    for v, i, p in diffs:
+        assert v <= tol, f"{label}: request {i}, position {p} (the first wrong one): |diff| {v:.3e} > {tol:.3e}"
+
+
+def check_request(cfg, tensors, tokens, got_rows, dtype, label=""):
+    check_requests(cfg, tensors, [(tokens, got_rows)], dtype, label)
 
 
 def run_cuts(engine, tokens, cuts, graphs=False):
