@@ -406,3 +406,317 @@ def test_head_kernel_for_values_that_are_the_keys(dtype, H, G, dim, rdims, lens)
             pg.put(want_v, b, p, [u[t, H:]])
     assert float((kc.cpu().double() - want_k).abs().max()) <= tol
     assert float((vc.cpu().double() - want_v).abs().max()) <= tol * 3
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("d", [40, 50, 1032])
+def test_mixes_with_the_token_before(dtype, d):
+    """All five mixes; a portion's first token reads the slot's last input, whichever tile it falls into; the lists by
+    which a grouped product takes the first four."""
+    from transformer_b200.csrc import lib
+    td, sfx = _td(dtype)
+    g = torch.Generator().manual_seed(d)
+    mu = torch.rand(5, d, generator=g)
+    size = lib.decay_state_size(2, 6, d)
+    state = torch.randn(7, size, generator=g)
+    d_mu, d_state = mu.cuda(), state.cuda()
+    for lens in ([1, 1, 1], [3, 1, 5], [130, 7, 190]):
+        nt = sum(lens)
+        slots = [4, 0, 6]
+        x = torch.randn(nt, d, generator=g).to(td)
+        pg = _Pages([0] * 3, lens, g)
+        out = torch.empty(5, nt, d, dtype=td, device="cuda")
+        offsets, groups = _ints([0] * 5), _ints([9] * (4 * nt))
+        d_x, d_slots = x.cuda(), _ints(slots)
+        lib.call("tb_shift_mix_" + sfx, lib.ptr(d_x), lib.ptr(d_mu), lib.ptr(d_state), size, 2 * 6 * 6, lib.ptr(out),
+                 lib.ptr(offsets), lib.ptr(groups), 4, lib.ptr(pg.tok_seq), lib.ptr(pg.seq_start), lib.ptr(d_slots), nt, d)
+        torch.cuda.synchronize()
+        before = torch.cat([torch.cat([state[s, 72:72 + d][None].double(), x[a:b - 1].double()])
+                            for s, a, b in zip(slots, pg.starts, pg.starts[1:])])
+        want = x.double()[None] + (before - x.double())[None] * mu.double()[:, None]
+        assert float((out.cpu().double() - want).abs().max()) <= (1e-5 if dtype == "float32" else 3e-2)
+        assert offsets.cpu().tolist() == [j * nt for j in range(5)]
+        assert groups.cpu().tolist() == [j for j in range(4) for _ in range(nt)]
+
+
+class _Memory:
+    """The recurrence's kernels over a batch in slots, carried from step to step, beside the plain recurrence."""
+
+    def __init__(self, dtype, H, dim, rank, width, seed):
+        from transformer_b200.csrc import lib
+        self.lib, (self.td, self.sfx) = lib, _td(dtype)
+        self.H, self.dim, self.rank, self.width = H, dim, rank, width
+        g = self.g = torch.Generator().manual_seed(seed)
+        hd = H * dim
+        self.w2 = (torch.randn(hd, rank, generator=g) * rank ** -0.5).to(self.td)
+        self.w0, self.u = torch.rand(hd, generator=g) * 4 - 4, torch.randn(H, dim, generator=g)
+        self.norm = torch.rand(hd, generator=g) + 0.5
+        size = lib.decay_state_size(H, dim, width)
+        self.pitch = size
+        self.state = torch.zeros(6, size, device="cuda")
+        self.seen = {}                      # slot -> lists of r, k, v, dec (plain, float64)
+
+    def open(self, slot):
+        self.state[slot].zero_()
+        self.seen[slot] = None
+
+    def step(self, slots, lens, make=None, single=False):
+        """One step; returns (engine rows [nt, H, dim] before the gate's effect is taken off, plain rows)."""
+        lib, H, dim, rank, td = self.lib, self.H, self.dim, self.rank, self.td
+        nt, hd = sum(lens), H * dim
+        z = torch.randn(4, nt, hd, generator=self.g)
+        a = torch.randn(nt, rank, generator=self.g)
+        if make is not None:
+            make(z.view(4, nt, H, dim), a)
+        z = z.to(td)
+        x = torch.randn(nt, self.width, generator=self.g).to(td)
+        starts = [0]
+        for n in lens:
+            starts.append(starts[-1] + n)
+        dev = lambda t: t.cuda()
+        d_z, d_a, d_x, d_w0, d_u, d_norm = map(dev, (z, a, x, self.w0, self.u, self.norm))
+        d_start, d_slots = _ints(starts), _ints(slots)
+        ldy = hd + 8
+        y = torch.full((nt, ldy), 3.0, dtype=td, device="cuda")
+        if single:
+            d_w2 = self.w2.cuda()
+            lib.call("tb_decay_step_" + self.sfx, lib.ptr(d_z), lib.ptr(d_x), self.width, lib.ptr(d_a), rank, lib.ptr(d_w2),
+                     lib.ptr(d_w0), lib.ptr(d_u), lib.ptr(d_norm), 1e-5, lib.ptr(self.state), self.pitch, lib.ptr(y), ldy,
+                     lib.ptr(d_start), lib.ptr(d_slots), nt, len(slots), H, dim, rank)
+        else:
+            half = (rank + 3) // 4 * 4
+            wide = rank if td == torch.float32 else 2 * half
+            th = torch.empty(nt, wide, dtype=td, device="cuda")
+            lib.call("tb_decay_tanh_" + self.sfx, lib.ptr(d_a), rank, lib.ptr(th), nt, rank, wide)
+            t64 = th.double().cpu()
+            got_tanh = t64[:, :rank] if td == torch.float32 else t64[:, :rank] + t64[:, half:half + rank]
+            assert float((got_tanh - torch.tanh(a.double())).abs().max()) <= (1e-6 if td == torch.float32 else 1e-5)
+            pre = (got_tanh @ self.w2.double().T).float().cuda()
+            rec = torch.empty(nt, H, lib.decay_record_size(dim), device="cuda")
+            vals = torch.empty(nt, H, lib.decay_value_pitch(dim), device="cuda")
+            o = torch.empty(nt, hd, device="cuda")
+            lib.call("tb_decay_prep_" + self.sfx, lib.ptr(d_z), lib.ptr(pre), lib.ptr(d_w0), lib.ptr(d_u), lib.ptr(rec),
+                     lib.ptr(vals), nt, H, dim)
+            lib.call("tb_decay_scan_" + self.sfx, lib.ptr(rec), lib.ptr(vals), lib.ptr(self.state), self.pitch, lib.ptr(o),
+                     lib.ptr(d_x), self.width, lib.ptr(d_start), lib.ptr(d_slots), nt, len(slots), H, dim)
+            lib.call("tb_mlstm_out_" + self.sfx, lib.ptr(o), lib.ptr(d_z[3]), hd, lib.ptr(d_norm), lib.ptr(y), nt, H, dim,
+                     1e-5, 1, ldy)
+        torch.cuda.synchronize()
+        dec = torch.exp(-torch.exp(torch.tanh(a.double()) @ self.w2.double().T + self.w0.double()))
+        want = torch.empty(nt, hd, dtype=torch.float64)
+        for b, s in enumerate(slots):
+            lo, hi = starts[b], starts[b + 1]
+            new = [t[lo:hi].double().view(hi - lo, H, dim) for t in (z[0], z[1], z[2], dec)]
+            old = self.seen[s]
+            self.seen[s] = new if old is None else [torch.cat([p, q]) for p, q in zip(old, new)]
+            full = FP.recurrence(*self.seen[s], self.u.double())[-(hi - lo):]
+            want[lo:hi] = FP.rms(full, 1e-5).reshape(hi - lo, hd) * self.norm.double() * FP.silu(z[3, lo:hi].double())
+            last = self.state[s, H * dim * dim:H * dim * dim + self.width].cpu()
+            assert torch.equal(last, x[hi - 1].float()), "the slot's last input"
+        got = y.cpu()
+        assert bool((got[:, hd:] == 3.0).all()), "entries beside the heads' were written"
+        return got[:, :hd].double(), want
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H, dim, rank", [(2, 64, 16), (1, 128, 64), (3, 7, 5), (2, 33, 12), (1, 256, 8), (4, 16, 8), (2, 96, 24)])
+def test_memory_carried_over_prompts_portions_and_single_tokens(dtype, H, dim, rank):
+    m = _Memory(dtype, H, dim, rank, 50, H + dim)
+    tol = 1e-3 if dtype == "float32" else 4e-2
+    for s in (3, 1, 5):
+        m.open(s)
+    plan = [([3, 1, 5], [17, 1, 40], False), ([3, 1, 5], [1, 1, 1], True), ([5, 3], [8, 2], False), ([1], [1], True),
+            ([1, 3], [23, 1], False), ([5, 1, 3], [1, 1, 1], True), ([3], [1], False)]
+    for i, (slots, lens, single) in enumerate(plan):
+        got, want = m.step(slots, lens, single=single)
+        scale = max(1.0, float(want.abs().max()))
+        assert float((got - want).abs().max()) <= tol * scale, f"step {i}: {float((got - want).abs().max()):.3e} of {scale:.2f}"
+    m.open(3)                               # the slot again, for another sequence
+    got, want = m.step([3], [9])
+    assert float((got - want).abs().max()) <= tol * max(1.0, float(want.abs().max())), "a slot used again"
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("single", [False, True])
+def test_memory_gives_back_what_was_written_long_ago(dtype, single):
+    """One strong write under key channel 5 whose decay is next to none, 300 tokens that write elsewhere, then a question
+    for that channel, in another step and in a used slot: the answer is the value that was written, whatever the gates."""
+    H, dim, rank = 2, 64, 8
+    m = _Memory(dtype, H, dim, rank, 40, 7)
+    m.w2.zero_()
+    m.w0 = torch.full((H * dim,), -1.0)
+    m.w0.view(H, dim)[:, 5] = -12.0         # keeps
+    m.open(2)
+    m.step([2], [30])
+    m.open(2)
+    value = torch.randn(H, dim, generator=m.g)
+
+    def write(z, a):
+        z[1] = 0
+        z[1, 0, :, 5], z[2, 0] = 4.0, value
+
+    def elsewhere(z, a):
+        z[1, :, :, 5] = 0
+
+    def ask(z, a):
+        z[0] = 0
+        z[0, :, :, 5], z[1], z[3] = 1.0, 0, 2.0
+
+    m.step([2], [1], write, single=single)
+    m.step([2], [300], elsewhere)
+    got, want = m.step([2], [1], ask, single=single)
+    tol = 1e-3 if dtype == "float32" else 4e-2
+    assert float((got - want).abs().max()) <= tol * float(want.abs().max())
+    v = value.to(m.td).double()
+    direct = FP.rms(v * 4.0, 0.0).reshape(-1) * m.norm.double() * FP.silu(torch.tensor(2.0, dtype=torch.float64))
+    assert float((got[0] - direct).abs().max()) <= 5e-2 * float(direct.abs().max())
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("d", [48, 50, 192, 4096, 6008, 13000])
+def test_stream_norm_in_all_its_forms(dtype, d):
+    """x <- y = N(alpha x + u): the delta a tensor or experts' rows; with and without what rides along (the table's
+    experts, equal weights, the shared expert's gate from the row as stored)."""
+    from transformer_b200.csrc import lib
+    td, sfx = _td(dtype)
+    g = torch.Generator().manual_seed(d)
+    n, k, terms, vocab = 6, 3, 4, 11
+    x0, delta = torch.randn(n, d, generator=g) * 2 + 0.5, (torch.randn(n, d, generator=g) * 3 + 1).to(td)
+    w, b = torch.rand(d, generator=g) + 0.5, torch.randn(d, generator=g)
+    ey, tw = torch.randn(n * terms, d, generator=g).to(td), torch.rand(n, terms, generator=g)
+    at = torch.randperm(n * terms, generator=g).to(torch.int32)
+    tok = torch.randint(0, vocab, (n,), generator=g).to(torch.int32)
+    table = torch.randint(0, 99, (vocab, k), generator=g).to(torch.int32)
+    gw = (torch.randn(d, generator=g) * d ** -0.5).to(td)
+    dv = [t.cuda() for t in (delta, w, b, ey, tw, at, tok, table, gw)]
+    d_delta, d_w, d_b, d_ey, d_tw, d_at, d_tok, d_table, d_gw = dv
+    for rows in (False, True):
+        for ride in ("nothing", "table", "table and gate"):
+            x, y = x0.clone().cuda(), torch.empty(n, d, dtype=td, device="cuda")
+            kk = k + (ride == "table and gate")
+            idx, wts = torch.full((n, k), -1, dtype=torch.int32, device="cuda"), torch.full((n, kk), -1.0, device="cuda")
+            pick = (0, 0, 0, 0, 0, 0) if ride == "nothing" else \
+                (lib.ptr(d_tok), lib.ptr(d_table), lib.ptr(d_gw) if kk > k else 0, lib.ptr(idx), lib.ptr(wts), k)
+            lib.call("tb_renew_layernorm_" + sfx, lib.ptr(x), 0 if rows else lib.ptr(d_delta), lib.ptr(d_ey) if rows else 0,
+                     lib.ptr(d_at) if rows else 0, lib.ptr(d_tw) if rows else 0, terms if rows else 0, 1.75, lib.ptr(d_w),
+                     lib.ptr(d_b), 1e-5, lib.ptr(y), n, d, *pick)
+            torch.cuda.synchronize()
+            u = torch.stack([sum(tw[t, j].double() * ey[at[t * terms + j]].double() for j in range(terms)) for t in range(n)]) \
+                if rows else delta.double()
+            want = FP.layer_norm(1.75 * x0.double() + u, w.double(), b.double(), 1e-5)
+            assert float((x.cpu().double() - want).abs().max()) < 3e-5, "the stream itself is float"
+            assert torch.equal(y.cpu(), x.cpu().to(td)), "the rows are the stream, rounded once"
+            if ride == "nothing":
+                continue
+            assert torch.equal(idx.cpu(), table[tok.long()])
+            assert float((wts[:, :k].cpu() - 1.0 / k).abs().max()) < 1e-7
+            if kk > k:
+                gate = torch.sigmoid(y.cpu().double() @ gw.double())
+                assert float((wts[:, k].cpu().double() - gate).abs().max()) < 1e-5
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_terms_and_lists_of_experts_with_a_shared_one(dtype):
+    from transformer_b200.csrc import lib
+    td, sfx = _td(dtype)
+    g = torch.Generator().manual_seed(1)
+    for nt, k, E, d in ((1, 1, 3, 40), (700, 2, 5, 50), (40, 4, 4, 128)):
+        x, gw = torch.randn(nt, d, generator=g).to(td), (torch.randn(d, generator=g) * d ** -0.5).to(td)
+        tok = torch.randint(0, 9, (nt,), generator=g).to(torch.int32)
+        table = torch.stack([torch.randperm(E, generator=g)[:k] for _ in range(9)]).to(torch.int32)
+        w_in = torch.rand(nt, k, generator=g)
+        d_x, d_gw, d_tok, d_table, d_win = x.cuda(), gw.cuda(), tok.cuda(), table.cuda(), w_in.cuda()
+        idx, wts = torch.zeros(nt, k, dtype=torch.int32, device="cuda"), torch.zeros(nt, k + 1, device="cuda")
+        lib.call("tb_moe_terms_" + sfx, lib.ptr(d_x), lib.ptr(d_gw), lib.ptr(d_tok), lib.ptr(d_table), 0, lib.ptr(idx),
+                 lib.ptr(wts), nt, d, k)
+        gate = torch.sigmoid(x.double() @ gw.double())
+        assert torch.equal(idx.cpu(), table[tok.long()]) and float((wts[:, :k].cpu() - 1 / k).abs().max()) < 1e-7
+        assert float((wts[:, k].cpu().double() - gate).abs().max()) < 1e-5
+        lib.call("tb_moe_terms_" + sfx, lib.ptr(d_x), 0, 0, 0, lib.ptr(d_win), 0, lib.ptr(wts), nt, d, k)
+        assert torch.equal(wts.view(-1)[:nt * k].cpu(), w_in.view(-1))
+        M = nt * k
+        off, st, at = _ints([0] * (E + 1)), _ints([0] * M), _ints([-1] * (nt * (k + 1)))
+        lib.call("tb_moe_dispatch_shared", lib.ptr(idx), lib.ptr(off), lib.ptr(st), lib.ptr(at), M, k, E)
+        off, st, at, ex = off.cpu(), st.cpu(), at.cpu().view(nt, k + 1), idx.cpu()
+        assert at[:, k].tolist() == [M + t for t in range(nt)] and sorted(at[:, :k].reshape(-1).tolist()) == list(range(M))
+        for t in range(nt):
+            for j in range(k):
+                r, e = int(at[t, j]), int(ex[t, j])
+                assert int(off[e]) <= r < int(off[e + 1]) and int(st[r]) == t
+
+
+def test_tanh_gelu_pair_in_every_product():
+    from transformer_b200.parts.linear import GELU_TANH, gemm_simt, gemm_skinny, gemm_tc
+    g = torch.Generator().manual_seed(0)
+    for M, K, N in ((5, 64, 40), (300, 128, 96)):
+        a, w = torch.randn(M, K, generator=g) * 3, torch.randn(2 * N, K, generator=g) * K ** -0.5
+
+        def want(a, w):
+            p = a.double() @ w.double().T
+            return FP.gelu_tanh(p[:, :N]) * p[:, N:]
+
+        out = torch.empty(M, N, device="cuda")
+        d_a, d_w = a.cuda(), w.cuda()
+        gemm_simt(d_a, d_w, out, out_kind=2, glu=GELU_TANH)
+        ref = want(a, w)
+        assert float((out.cpu().double() - ref).abs().max()) <= 2e-5 * float(ref.abs().max())
+        ab, wb = a.bfloat16(), w.bfloat16()
+        d_a, d_w, ref = ab.cuda(), wb.cuda(), want(ab, wb)
+        for product in (gemm_skinny, gemm_tc):
+            out = torch.empty(M, N, dtype=torch.bfloat16, device="cuda")
+            assert product(d_a, d_w, out, out_kind=2, glu=GELU_TANH)
+            torch.cuda.synchronize()
+            assert float((out.cpu().double() - ref).abs().max()) <= 2.0 ** -7 * float(ref.abs().max()), product.__name__
+
+
+def test_a_shared_expert_beside_a_router(tmp_path):
+    """The shared expert goes with any choice of experts: a pre-norm block with a softmax router and a shared expert, a
+    prompt and single tokens against each other and against the same layer computed in torch."""
+    from transformer_b200.architectures.generic import plan_from_spec
+    from transformer_b200.engine import Engine
+    from transformer_b200.parts.spec import LayerSpec, ModelSpec, PartSpec, RunEntry
+    from transformer_b200.weights.random_init import random_device_weights
+    d, E, k, di, sh, V = 64, 4, 2, 48, 40, 60
+    norm = PartSpec.of("rmsnorm", width=d, eps=1e-6)
+    att = PartSpec.of("attention", width=d, nh=2, nkvh=1, dh=32, position=PartSpec.of("rope", dh=32, theta=1e4, positions=256))
+    ff = PartSpec.of("moe", width=d, di=di, nexp=E, nexp_use=k, shared_di=sh)
+    spec = ModelSpec(width=d, vocab=V, max_context=256, layers=(LayerSpec(att, ff, norm, norm),), order=(RunEntry(0),),
+                     embedding=PartSpec.of("lookup", vocab=V, width=d), final_norm=norm,
+                     head=PartSpec.of("linear", vocab=V, width=d, tied=False))
+    dev = torch.device("cuda:0")
+    rules = plan_from_spec(spec)
+    weights = random_device_weights(rules, 3, torch.float32, dev, 0.3)
+    engine = Engine(spec, weights, torch.float32, dev, max_tokens=512)
+    tokens = random_prompts(V, [70], 1)[0]
+    whole = engine.step([engine.open()], [tokens], [list(range(70))]).cpu()
+    slot = engine.open()
+    engine.step([slot], [tokens[:60]])
+    for p in range(60, 70):
+        assert float((engine.step([slot], [[tokens[p]]]).cpu()[0] - whole[p]).abs().max()) < 1e-3
+    seen = {}
+    part = engine.layers[0].feed_forward
+    x = torch.randn(9, d, generator=torch.Generator().manual_seed(5))
+
+    class Ctx:
+        tok_ids = None
+        decode = False
+
+        def scratch(self, name, shape, dtype, zero=False):
+            return seen.setdefault(name, torch.zeros(shape, dtype=dtype, device=dev))
+
+        def record(self, *a):
+            pass
+    got = part.forward(Ctx(), x.cuda(), None)
+    out = torch.empty(9, d, device=dev)
+    from transformer_b200.parts.feed_forward import sum_weighted_rows
+    sum_weighted_rows(got, out)
+    W = {n: t.double().cpu() for n, t in part.weights.items()}
+    want = torch.zeros(9, d, dtype=torch.float64)
+    for t in range(9):
+        h = x[t].double()
+        top = torch.topk(W["router"] @ h, k)
+        for a, e in zip(torch.softmax(top.values, 0), top.indices.tolist()):
+            want[t] += a * (W["wd"][e] @ (FP.silu(W["wgu"][e, :di] @ h) * (W["wgu"][e, di:] @ h)))
+        s = W["shared_wd"] @ (FP.silu(W["shared_wgu"][:sh] @ h) * (W["shared_wgu"][sh:] @ h))
+        want[t] += torch.sigmoid(W["shared_gate"][0] @ h) * s
+    assert float((out.cpu().double() - want).abs().max()) <= 1e-4 * float(want.abs().max())
