@@ -492,12 +492,11 @@ class _Memory:
             got_tanh = t64[:, :rank] if td == torch.float32 else t64[:, :rank] + t64[:, half:half + rank]
             assert float((got_tanh - torch.tanh(a.double())).abs().max()) <= (1e-6 if td == torch.float32 else 1e-5)
             pre = (got_tanh @ self.w2.double().T).float().cuda()
-            rec = torch.empty(nt, H, lib.decay_record_size(dim), device="cuda")
-            vals = torch.empty(nt, H, lib.decay_value_pitch(dim), device="cuda")
+            rec = torch.empty(H, nt, lib.decay_record_size(dim), device="cuda")
             o = torch.empty(nt, hd, device="cuda")
             lib.call("tb_decay_prep_" + self.sfx, lib.ptr(d_z), lib.ptr(pre), lib.ptr(d_w0), lib.ptr(d_u), lib.ptr(rec),
-                     lib.ptr(vals), nt, H, dim)
-            lib.call("tb_decay_scan_" + self.sfx, lib.ptr(rec), lib.ptr(vals), lib.ptr(self.state), self.pitch, lib.ptr(o),
+                     nt, H, dim)
+            lib.call("tb_decay_scan_" + self.sfx, lib.ptr(rec), lib.ptr(self.state), self.pitch, lib.ptr(o),
                      lib.ptr(d_x), self.width, lib.ptr(d_start), lib.ptr(d_slots), nt, len(slots), H, dim)
             lib.call("tb_mlstm_out_" + self.sfx, lib.ptr(o), lib.ptr(d_z[3]), hd, lib.ptr(d_norm), lib.ptr(y), nt, H, dim,
                      1e-5, 1, ldy)

@@ -12,7 +12,8 @@
 //
 //   shift_mix_kernel    all mixes of a token at once, and the group lists of the product that follows (a matrix per mix)
 //   decay_tanh_kernel   prompts: tanh(a) for the product with W2
-//   decay_prep_kernel   prompts: decays and bonuses; one float record per (token, head) for the scan, r | k | w | bonus
+//   decay_prep_kernel   prompts: decays and bonuses; one float record per (token, head) for the scan, r | k | w | v | bonus,
+//                       those of a head one behind the other
 //   decay_scan_kernel   prompts: the recurrence token by token, a block = a sequence x a head x some columns of S, whose
 //                       rows are split over adjacent lanes, in registers; the lanes' sums meet only in the output, so
 //                       no token waits for another's reduction
@@ -20,7 +21,7 @@
 //                       registers, the head's norm and the gate in one kernel
 // Everything that enters the recurrence is float on both paths; x, r, k, v and the gate have the activations' type.
 #include "common.cuh"
-#include "attention_prefill.cuh"        // cp_async16, cp_async_commit, cp_async_wait
+#include "tc_common.cuh"                // bulk copies, barriers with bounded waits
 
 constexpr int DM_MIXES = 5;             // r, k, v, gate, decay
 constexpr int DM_TOK = 8;               // tokens of a stage of the scan
@@ -28,8 +29,7 @@ constexpr int DM_STAGES = 4;            // stages in flight or in use
 constexpr int DM_SCAN = 128;            // threads of a scan block
 
 __host__ __device__ inline int dm_rows(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
-__host__ __device__ inline int dm_record(int dim) { return 3 * dm_rows(dim) + 4; }
-__host__ __device__ inline int dm_vpitch(int dim) { return (dim + 31) / 32 * 32; }
+__host__ __device__ inline int dm_record(int dim) { return 4 * dm_rows(dim) + 4; }
 __host__ __device__ inline long long dm_state(int H, int dim, int width) { return ((long long)H * dim * dim + width + 3) / 4 * 4; }
 
 // ---- the mixes ---------------------------------------------------------------------------------------------
@@ -190,8 +190,7 @@ struct DecayArgs {
     const float* pre;       // [nt, H dim]  W2 tanh(.)
     const float* w0;        // [H dim]
     const float* u;         // [H dim]
-    float* rec;             // [nt, H, dm_record]
-    float* vals;            // [nt, H, dm_vpitch]
+    float* rec;             // [H, nt, dm_record]
     int nt, H, dim;
 };
 
@@ -205,13 +204,12 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DecayArgs p) {
     const int row = blockIdx.x * 8 + (threadIdx.x >> 5);
     if (row >= p.nt * p.H) return;
     const int t = row / p.H, h = row - t * p.H, dim = p.dim, hd = p.H * dim;
-    const int DP = dm_rows(dim), VP = dm_vpitch(dim);
-    float* rec = p.rec + (size_t)row * dm_record(dim);
-    float* vals = p.vals + (size_t)row * VP;
+    const int DP = dm_rows(dim);
+    float* rec = p.rec + ((size_t)h * p.nt + t) * dm_record(dim);
     const T* z = static_cast<const T*>(p.z) + (size_t)t * hd + h * dim;
     const size_t part = (size_t)p.nt * hd;
     float bonus = 0.f;
-    for (int c = lane * V; c < max(DP, VP); c += 32 * V) {
+    for (int c = lane * V; c < DP; c += 32 * V) {
         float r[V], k[V], v[V], w[V];
 #pragma unroll
         for (int e = 0; e < V; ++e) {
@@ -232,28 +230,26 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DecayArgs p) {
                 bonus += r[e] * u[e] * k[e];
             }
         }
-        if (c < DP) {
-            dm_store<V>(rec + c, r);
-            dm_store<V>(rec + DP + c, k);
-            dm_store<V>(rec + 2 * DP + c, w);
-        }
-        if (c < VP) dm_store<V>(vals + c, v);
+        dm_store<V>(rec + c, r);
+        dm_store<V>(rec + DP + c, k);
+        dm_store<V>(rec + 2 * DP + c, w);
+        dm_store<V>(rec + 3 * DP + c, v);
     }
     bonus = warp_sum(bonus);
-    if (lane < 4) rec[3 * DP + lane] = lane == 0 ? bonus : 0.f;
+    if (lane < 4) rec[4 * DP + lane] = lane == 0 ? bonus : 0.f;
 }
 
 // ---- the scan ------------------------------------------------------------------------------------------------
 struct DecayScanArgs {
     const float* rec;
-    const float* vals;
     float* state;           // [slots, pitch]
+    int* error;             // set by a wait that runs out
     float* out;             // [nt, H dim]
     const void* x;          // [nt, width]: a sequence's last row becomes its state's last input
     const int* seq_start;
     const int* slots;
     long long pitch;
-    int H, dim, width;
+    int nt, H, dim, width;
 };
 
 // two floats in one register pair, and the hardware's packed multiply-add on them
@@ -273,7 +269,8 @@ __device__ __forceinline__ F2 mul2(F2 a, F2 b) {
 }
 
 // RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): DM_SCAN / SPLIT * C columns a
-// block.  The records of DM_TOK tokens at a time are copied to shared memory by cp.async, DM_STAGES - 1 stages ahead.  A
+// block.  The records of DM_TOK tokens at a time are one bulk copy to shared memory,
+// DM_STAGES - 1 stages ahead.  A
 // token needs no reduction: every lane keeps its rows' share of the outputs of a whole stage, and the DM_TOK * C shares
 // are then summed over the column's lanes so that each lane ends with some of the sums (fewer shuffles than sums).
 template <typename T, int RPT, int SPLIT, int C>
@@ -281,19 +278,17 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
     pdl_sync();
     constexpr int DP = RPT * SPLIT;
     constexpr int COLS = DM_SCAN / SPLIT * C;
-    constexpr int PER = 3 * DP + 4;
-    constexpr int ROW = PER + COLS;
-    constexpr int ROW4 = ROW / 4;
+    constexpr int ROW = 4 * DP + 4;                     // a record
     constexpr int NV = DM_TOK * C;
-    static_assert(NV % SPLIT == 0 && COLS % 4 == 0, "every lane ends with as many sums");
+    static_assert(NV % SPLIT == 0, "every lane ends with as many sums");
     extern __shared__ __align__(16) float dm_sm[];      // [DM_STAGES][DM_TOK][ROW]
+    __shared__ __align__(8) unsigned long long bars[DM_STAGES];
     const int b = blockIdx.x, h = blockIdx.y;
     const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT * C;
     const int col0 = blockIdx.z * COLS, col = col0 + cl;
     const int dim = a.dim, H = a.H;
     const int t0 = a.seq_start[b], t1 = a.seq_start[b + 1];
     if (t0 >= t1) return;
-    const int VP = dm_vpitch(dim);
     float* slot = a.state + (size_t)a.slots[b] * a.pitch;
     float* S = slot + (size_t)h * dim * dim;
     F2 s[C][RPT / 2];                                   // rows 2i, 2i + 1 of this lane's
@@ -305,16 +300,21 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
             s[c][i].f.x = (r < dim && col + c < dim) ? S[(size_t)r * dim + col + c] : 0.f;
             s[c][i].f.y = (r + 1 < dim && col + c < dim) ? S[(size_t)(r + 1) * dim + col + c] : 0.f;
         }
-    auto issue = [&](int ts) {
-        const int n = min(DM_TOK, t1 - ts);
-        float* to = dm_sm + (size_t)((ts - t0) / DM_TOK % DM_STAGES) * (DM_TOK * ROW);
-        for (int idx = tid; idx < n * ROW4; idx += DM_SCAN) {
-            const int tt = idx / ROW4, e4 = idx - tt * ROW4;
-            // columns behind the padded row of values are left alone: no column of the head reads them
-            if (e4 >= PER / 4 && col0 + (e4 - PER / 4) * 4 >= VP) continue;
-            const float* src = e4 < PER / 4 ? a.rec + ((size_t)(ts + tt) * H + h) * PER + e4 * 4
-                                            : a.vals + ((size_t)(ts + tt) * H + h) * VP + col0 + (e4 - PER / 4) * 4;
-            cp_async16((uint32_t)__cvta_generic_to_shared(to + tt * ROW + e4 * 4), src);
+    const float* rec = a.rec + (size_t)h * a.nt * ROW;
+    const uint32_t bar0 = smem_u32(bars);
+    if (tid == 0) {
+        for (int q = 0; q < DM_STAGES; ++q) mbar_init(bar0 + 8u * q, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    const int stages = (t1 - t0 + DM_TOK - 1) / DM_TOK;
+    auto issue = [&](int q) {
+        const int ts = t0 + q * DM_TOK, n = min(DM_TOK, t1 - ts);
+        float* to = dm_sm + (size_t)(q % DM_STAGES) * (DM_TOK * ROW);
+        if (tid == 0) {
+            const uint32_t bytes = (uint32_t)(n * ROW) * sizeof(float);
+            mbar_expect_tx(bar0 + 8u * (q % DM_STAGES), bytes);
+            bulk_load(smem_u32(to), rec + (size_t)ts * ROW, bytes, bar0 + 8u * (q % DM_STAGES));
         }
         // tokens behind the last: nothing is written, nothing fades, nothing is read (so that a stage has no branches)
         for (int idx = n * ROW + tid; idx < DM_TOK * ROW; idx += DM_SCAN) {
@@ -322,17 +322,19 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
             to[idx] = e >= 2 * DP && e < 3 * DP ? 1.f : 0.f;
         }
     };
-#pragma unroll
-    for (int q = 0; q < DM_STAGES - 1; ++q) {
-        if (t0 + q * DM_TOK < t1) issue(t0 + q * DM_TOK);
-        cp_async_commit();
-    }
-    for (int ts = t0; ts < t1; ts += DM_TOK) {
-        cp_async_wait<DM_STAGES - 2>();
-        __syncthreads();            // this stage has landed for everyone, and everyone is done with the stage before
-        if (ts + (DM_STAGES - 1) * DM_TOK < t1) issue(ts + (DM_STAGES - 1) * DM_TOK);
-        cp_async_commit();
-        const float* stage = dm_sm + (size_t)((ts - t0) / DM_TOK % DM_STAGES) * (DM_TOK * ROW);
+    int issued = 0;
+    for (; issued < DM_STAGES - 1 && issued < stages; ++issued) issue(issued);
+    for (int st = 0; st < stages; ++st) {
+        const bool ok = mbar_wait(bar0 + 8u * (st % DM_STAGES), (st / DM_STAGES) & 1, a.error, 31);
+        // the stage has landed for everyone, and everyone is done with the stage before
+        if (!__syncthreads_and(ok)) {
+            if (tid == 0)
+                for (int q = st; q < issued; ++q) mbar_wait(bar0 + 8u * (q % DM_STAGES), (q / DM_STAGES) & 1, a.error, 32);
+            return;
+        }
+        if (issued < stages) issue(issued++);
+        const int ts = t0 + st * DM_TOK;
+        const float* stage = dm_sm + (size_t)(st % DM_STAGES) * (DM_TOK * ROW);
         const int n = min(DM_TOK, t1 - ts);
         float o[NV];
 #pragma unroll
@@ -341,7 +343,7 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
             F2 v[C], d[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                v[c].f.x = v[c].f.y = row[PER + cl + c];
+                v[c].f.x = v[c].f.y = row[3 * DP + min(col + c, DP - 1)];
                 d[c].f.x = d[c].f.y = 0.f;
             }
 #pragma unroll
@@ -380,7 +382,7 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
             const int idx = part * (NV / SPLIT) + j, tt = idx / C, c = idx % C;
             if (tt < n && col + c < dim) {
                 const float* row = stage + tt * ROW;
-                a.out[((size_t)(ts + tt) * H + h) * dim + col + c] = o[j] + row[3 * DP] * row[PER + cl + c];
+                a.out[((size_t)(ts + tt) * H + h) * dim + col + c] = o[j] + row[4 * DP] * row[3 * DP + col + c];
             }
         }
     }
@@ -404,7 +406,7 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
 template <typename T, int RPT, int SPLIT, int C>
 static int decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
     constexpr int COLS = DM_SCAN / SPLIT * C;
-    const size_t smem = (size_t)DM_STAGES * DM_TOK * (3 * RPT * SPLIT + 4 + COLS) * sizeof(float);
+    const size_t smem = (size_t)DM_STAGES * DM_TOK * (4 * RPT * SPLIT + 4) * sizeof(float);
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
         cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -420,11 +422,13 @@ static int decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t
 }
 
 template <typename T>
-static int decay_scan_launch(const DecayScanArgs& a, int nt, int B, cudaStream_t s) {
+static int decay_scan_launch(DecayScanArgs a, int B, cudaStream_t s) {
     if (B < 0 || a.H <= 0 || a.dim <= 0 || a.width <= 0 || a.pitch < dm_state(a.H, a.dim, a.width)) return TB_ERR_ARG;
     if (a.dim > 256) return TB_ERR_UNSUPPORTED;
     if (B == 0) return 0;
-    const bool early = nt <= 2 * B;
+    a.error = tc_error_ptr();
+    if (!a.error) return tb_last_error();
+    const bool early = a.nt <= 2 * B;
     switch (dm_rows(a.dim)) {
         case 16: return decay_scan_go<T, 4, 4, 1>(a, B, early, s);
         case 32: return decay_scan_go<T, 4, 8, 1>(a, B, early, s);
@@ -595,7 +599,6 @@ extern "C" {
 // Floats of state per slot.
 int tb_decay_state_size(int H, int dim, int width) { return (int)dm_state(H, dim, width); }
 int tb_decay_record_size(int dim) { return dm_record(dim); }
-int tb_decay_value_pitch(int dim) { return dm_vpitch(dim); }
 // out [5, nt, d]: the mixes of every token; offsets [groups + 1] and row_group [groups nt] (may be null): the lists by
 // which one grouped product multiplies the first `groups` of them with a matrix each.  `at`: where in a slot's state the
 // last input lies.
@@ -610,16 +613,15 @@ int tb_decay_value_pitch(int dim) { return dm_vpitch(dim); }
         return decay_tanh_launch<T>(a, lda, out, nt, rank, ldo, s);                                                   \
     }                                                                                                                 \
     int tb_decay_prep_##SFX(const void* z, const float* pre, const float* w0, const float* u, float* rec,             \
-                            float* vals, int nt, int H, int dim, cudaStream_t s) {                                    \
-        if (((uintptr_t)rec | (uintptr_t)vals) & 15) return TB_ERR_ARG;                                               \
-        return decay_prep_launch<T>(DecayArgs{z, pre, w0, u, rec, vals, nt, H, dim}, s);                              \
+                            int nt, int H, int dim, cudaStream_t s) {                                                 \
+        if ((uintptr_t)rec & 15) return TB_ERR_ARG;                                                                   \
+        return decay_prep_launch<T>(DecayArgs{z, pre, w0, u, rec, nt, H, dim}, s);                              \
     }                                                                                                                 \
-    int tb_decay_scan_##SFX(const float* rec, const float* vals, float* state, long long pitch, float* out,           \
-                            const void* x, int width, const int* seq_start, const int* slots, int nt, int B, int H,   \
-                            int dim, cudaStream_t s) {                                                                \
-        if (((uintptr_t)rec | (uintptr_t)vals) & 15) return TB_ERR_ARG;                                               \
-        return decay_scan_launch<T>(DecayScanArgs{rec, vals, state, out, x, seq_start, slots, pitch, H, dim, width},  \
-                                    nt, B, s);                                                                        \
+    int tb_decay_scan_##SFX(const float* rec, float* state, long long pitch, float* out, const void* x, int width,    \
+                            const int* seq_start, const int* slots, int nt, int B, int H, int dim, cudaStream_t s) {  \
+        if ((uintptr_t)rec & 15) return TB_ERR_ARG;                                                                   \
+        return decay_scan_launch<T>(DecayScanArgs{rec, state, nullptr, out, x, seq_start, slots, pitch, nt, H, dim,   \
+                                                  width}, B, s);                                                      \
     }                                                                                                                 \
     int tb_decay_step_##SFX(const void* z, const void* x, int width, const float* a, int lda, const void* w2,         \
                             const float* w0, const float* u, const float* norm, float eps, float* state,              \

@@ -87,8 +87,8 @@ _SIGNATURES: Dict[str, str] = {
     "tb_attention_window_mma_heads_bf16": "pppppppppppiiiiiiiiiiiiffipppifi",
     "tb_shift_mix_f32": "pppllpppipppii", "tb_shift_mix_bf16": "pppllpppipppii",
     "tb_decay_tanh_f32": "pipiii", "tb_decay_tanh_bf16": "pipiii",
-    "tb_decay_prep_f32": "ppppppiii", "tb_decay_prep_bf16": "ppppppiii",
-    "tb_decay_scan_f32": "ppplppippiiii", "tb_decay_scan_bf16": "ppplppippiiii",
+    "tb_decay_prep_f32": "pppppiii", "tb_decay_prep_bf16": "pppppiii",
+    "tb_decay_scan_f32": "pplppippiiii", "tb_decay_scan_bf16": "pplppippiiii",
     "tb_decay_step_f32": "ppipippppfplpippiiiii", "tb_decay_step_bf16": "ppipippppfplpippiiiii",
     "tb_post_add_layernorm_router_f32": "pppppippfipppfipiippppiii",
     "tb_post_add_layernorm_router_bf16": "pppppippfipppfipiippppiii",
@@ -112,7 +112,7 @@ class TapeMap(ctypes.Structure):
     _fields_ = [("base", ctypes.c_ulonglong), ("size", ctypes.c_ulonglong), ("delta", ctypes.c_longlong)]
 
 
-_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i", "tb_decay_value_pitch": "i",
+_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i",
               "tb_attention_window_mma_tile_tokens": "ii", "tb_delta_state_size": "iiiii", "tb_delta_record_size": "i", "tb_delta_scan_lanes": "i", "tb_delta_value_pitch": "i", "tb_mlstm_state_size": "ii", "tb_latent_attention_tile_tokens": "i", "tb_attention_tile_tokens": "ii", "tb_gemm_tc_status": "", "tb_attention_prefill_tile_tokens": "",
               "tb_attention_tc_tile_tokens": ""}
 
@@ -374,13 +374,15 @@ def kernel_status_async(host_int32: torch.Tensor) -> None:
 
 def _gave_up(code: int) -> str:
     """Which kernel family a wait code belongs to (1..5 tensor-core products, 11..17 tensor-core prompt
-    attention, 21..22 decode attention with the page ring)."""
+    attention, 21..27 decode attention with the page ring, 31..32 the decaying memory's scan)."""
     if 1 <= code <= 5:
         return "tensor-core matrix product"
     if 11 <= code <= 17:
         return "tensor-core prompt attention"
     if 21 <= code <= 22:
         return "decode attention"
+    if 31 <= code <= 32:
+        return "scan of the decaying memory"
     return "unknown kernel"
 
 
@@ -425,11 +427,6 @@ def decay_state_size(heads: int, dim: int, width: int) -> int:
 def decay_record_size(dim: int) -> int:
     """Floats of the record that the decaying memory's first kernel leaves the scan per (token, head)."""
     return library().tb_decay_record_size(dim)
-
-
-def decay_value_pitch(dim: int) -> int:
-    """Floats of a (token, head) row of values between the decaying memory's two kernels for prompts."""
-    return library().tb_decay_value_pitch(dim)
 
 
 def attention_window_mma_tile_tokens(nh: int, nkvh: int) -> int:

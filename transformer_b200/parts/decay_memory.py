@@ -98,16 +98,15 @@ class DecayMemory(Mixer):
                 lib.ptr(w["w0"]), lib.ptr(w["u"]), lib.ptr(w["norm"]), self.eps, lib.ptr(state), pitch, lib.ptr(rows),
                 rows.stride(0), lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, H, self.dim, self.rank):
             return
-        rec = ctx.scratch("decay.rec", (nt, H, lib.decay_record_size(self.dim)), torch.float32)
-        vals = ctx.scratch("decay.v", (nt, H, lib.decay_value_pitch(self.dim)), torch.float32)
+        rec = ctx.scratch("decay.rec", (H, nt, lib.decay_record_size(self.dim)), torch.float32)
         th = ctx.scratch("decay.tanh", (nt, self.tanh_width), self.dtype)
         lib.call("tb_decay_tanh_" + sfx, lib.ptr(a), self.rank, lib.ptr(th), nt, self.rank, self.tanh_width)
         pre = ctx.scratch("decay.pre", (nt, hd), torch.float32)
         matmul_nt(th, w["w2_tanh"], pre)                                    # float out
         lib.call("tb_decay_prep_" + sfx, lib.ptr(z), lib.ptr(pre), lib.ptr(w["w0"]), lib.ptr(w["u"]), lib.ptr(rec),
-                 lib.ptr(vals), nt, H, self.dim)
+                 nt, H, self.dim)
         o = ctx.scratch("decay.o", (nt, hd), torch.float32)
-        lib.call("tb_decay_scan_" + sfx, lib.ptr(rec), lib.ptr(vals), lib.ptr(state), pitch, lib.ptr(o), lib.ptr(x1), d,
+        lib.call("tb_decay_scan_" + sfx, lib.ptr(rec), lib.ptr(state), pitch, lib.ptr(o), lib.ptr(x1), d,
                  lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, H, self.dim)
         gate = z[3 * nt:]
         lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(gate), hd, lib.ptr(w["norm"]), lib.ptr(rows), nt, H, self.dim,
