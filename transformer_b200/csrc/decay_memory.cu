@@ -133,31 +133,23 @@ __device__ __forceinline__ void dm_store(float* p, const float (&f)[V]) {
 }
 
 // ---- decays ------------------------------------------------------------------------------------------------
-// w0 + W2 row . ta for DT tokens at once; ta [DT][rank] in shared memory
-template <typename T, int DT>
-__device__ __forceinline__ void decay_dot(const T* __restrict__ w2row, const float* ta, int rank, float base,
-                                          float (&acc)[DT]) {
-#pragma unroll
-    for (int p = 0; p < DT; ++p) acc[p] = base;
+// This lane's share of W2 row . ta: `parts` adjacent lanes take a row's pieces of eight (or entries) in turn.
+template <typename T>
+__device__ __forceinline__ float decay_dot(const T* __restrict__ w2row, const float* ta, int rank, int part, int parts) {
+    float acc = 0.f;
     if ((rank & 7) == 0) {
-        for (int q = 0; q < rank; q += 8) {
+#pragma unroll 4
+        for (int q = part * 8; q < rank; q += parts * 8) {
             float w[8];
             load8(w2row + q, w);
-#pragma unroll
-            for (int p = 0; p < DT; ++p) {
-                const float4 t0 = *reinterpret_cast<const float4*>(ta + p * rank + q);
-                const float4 t1 = *reinterpret_cast<const float4*>(ta + p * rank + q + 4);
-                acc[p] += w[0] * t0.x + w[1] * t0.y + w[2] * t0.z + w[3] * t0.w + w[4] * t1.x + w[5] * t1.y + w[6] * t1.z +
-                          w[7] * t1.w;
-            }
+            const float4 t0 = *reinterpret_cast<const float4*>(ta + q);
+            const float4 t1 = *reinterpret_cast<const float4*>(ta + q + 4);
+            acc += w[0] * t0.x + w[1] * t0.y + w[2] * t0.z + w[3] * t0.w + w[4] * t1.x + w[5] * t1.y + w[6] * t1.z + w[7] * t1.w;
         }
-        return;
+        return acc;
     }
-    for (int q = 0; q < rank; ++q) {
-        const float w = ldf(w2row + q);
-#pragma unroll
-        for (int p = 0; p < DT; ++p) acc[p] += w * ta[p * rank + q];
-    }
+    for (int q = part; q < rank; q += parts) acc += ldf(w2row + q) * ta[q];
+    return acc;
 }
 
 // tanh of the decay's first projection, ready for the product with W2: in the activations' type a value is stored as the
@@ -482,7 +474,7 @@ struct DecayStepArgs {
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) {
     constexpr int V = VEC ? 4 : 1;
-    constexpr int U = VEC ? 4 : 8;          // rows asked for together
+    constexpr int U = 8;                    // rows asked for together
     extern __shared__ __align__(16) float dm_sm[];
     const int b = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int dim = p.dim, hd = p.H * dim, rank4 = (p.rank + 3) / 4 * 4, dim4 = (dim + 3) / 4 * 4;
@@ -495,9 +487,8 @@ __global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) 
     float* o_s = v_s + dim4;                // [G][dim4]
     __shared__ float red[33];
     const int hc = h * dim + tid;
-    float w0 = 0.f, u = 0.f, nw = 0.f;
+    float u = 0.f, nw = 0.f;
     if (tid < dim) {                        // weights: nothing of the step writes them
-        w0 = p.w0[hc];
         u = p.u[hc];
         nw = p.norm[hc];
     }
@@ -506,6 +497,23 @@ __global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) 
     float* slot = p.state + (size_t)p.slots[b] * p.pitch;
     float* S = slot + (size_t)h * dim * dim;
     const T* z = static_cast<const T*>(p.z);
+    // the state's first rows are on their way while the decays are made
+    const int rg = tid / nc, c = (tid - rg * nc) * V;
+    float s[U][V];
+    auto fetch = [&](int r0) {
+#pragma unroll
+        for (int q = 0; q < U; ++q) {
+            const int r = r0 + q * G;
+            if (r >= dim) continue;
+            if constexpr (VEC) {
+                const float4 f = *reinterpret_cast<const float4*>(S + (size_t)r * dim + c);
+                s[q][0] = f.x; s[q][1] = f.y; s[q][2] = f.z; s[q][3] = f.w;
+            } else {
+                s[q][0] = S[(size_t)r * dim + c];
+            }
+        }
+    };
+    if (rg < G) fetch(rg);
     for (int q = tid; q < p.rank; q += 256) ta[q] = tanhf(p.a[(size_t)t * p.lda + q]);
     float bonus = 0.f, gate = 0.f;
     if (tid < dim) {
@@ -517,13 +525,16 @@ __global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) 
         bonus = r * u * k;
     }
     __syncthreads();
-    if (tid < dim) {
-        float acc[1];
-        decay_dot<T, 1>(static_cast<const T*>(p.w2) + (size_t)hc * p.rank, ta, p.rank, w0, acc);
-        w_s[tid] = expf(-expf(acc[0]));
+    {
+        // adjacent lanes share a channel's row of W2
+        const int parts = 256 / dm_rows(dim), ch = tid / parts, part = tid - ch * parts;
+        float acc = 0.f;
+        if (ch < dim)
+            acc = decay_dot<T>(static_cast<const T*>(p.w2) + (size_t)(h * dim + ch) * p.rank, ta, p.rank, part, parts);
+        for (int o = parts >> 1; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (ch < dim && part == 0) w_s[ch] = expf(-expf(acc + p.w0[h * dim + ch]));
     }
     bonus = block_sum(bonus, red);          // (and everyone's part of w_s is there)
-    const int rg = tid / nc, c = (tid - rg * nc) * V;
     if (rg < G) {
         float acc[V], v[V];
 #pragma unroll
@@ -532,19 +543,7 @@ __global__ void __launch_bounds__(256) decay_step_kernel(const DecayStepArgs p) 
             v[e] = v_s[c + e];
         }
         for (int r0 = rg; r0 < dim; r0 += G * U) {
-            float s[U][V];
-#pragma unroll
-            for (int q = 0; q < U; ++q) {
-                const int r = r0 + q * G;
-                if (r < dim) {
-                    if constexpr (VEC) {
-                        const float4 f = *reinterpret_cast<const float4*>(S + (size_t)r * dim + c);
-                        s[q][0] = f.x; s[q][1] = f.y; s[q][2] = f.z; s[q][3] = f.w;
-                    } else {
-                        s[q][0] = S[(size_t)r * dim + c];
-                    }
-                }
-            }
+            if (r0 != rg) fetch(r0);
 #pragma unroll
             for (int q = 0; q < U; ++q) {
                 const int r = r0 + q * G;
