@@ -518,7 +518,7 @@ class _Memory:
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H, dim, rank", [(2, 64, 16), (1, 128, 64), (3, 7, 5), (2, 33, 12), (1, 256, 8), (4, 16, 8), (2, 96, 24)])
+@pytest.mark.parametrize("H, dim, rank", [(2, 64, 16), (1, 128, 64), (3, 7, 5), (2, 33, 12), (1, 256, 8), (4, 16, 8), (2, 96, 24), (24, 64, 8), (12, 128, 8)])
 def test_memory_carried_over_prompts_portions_and_single_tokens(dtype, H, dim, rank):
     m = _Memory(dtype, H, dim, rank, 50, H + dim)
     tol = 1e-3 if dtype == "float32" else 4e-2

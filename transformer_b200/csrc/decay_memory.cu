@@ -24,8 +24,6 @@
 #include "tc_common.cuh"                // bulk copies, barriers with bounded waits
 
 constexpr int DM_MIXES = 5;             // r, k, v, gate, decay
-constexpr int DM_TOK = 8;               // tokens of a stage of the scan
-constexpr int DM_STAGES = 4;            // stages in flight or in use
 constexpr int DM_SCAN = 128;            // threads of a scan block
 
 __host__ __device__ inline int dm_rows(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
@@ -261,20 +259,20 @@ __device__ __forceinline__ F2 mul2(F2 a, F2 b) {
 }
 
 // RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): DM_SCAN / SPLIT * C columns a
-// block.  The records of DM_TOK tokens at a time are one bulk copy to shared memory,
-// DM_STAGES - 1 stages ahead.  A
-// token needs no reduction: every lane keeps its rows' share of the outputs of a whole stage, and the DM_TOK * C shares
+// block.  The records of TOK tokens at a time are one bulk copy to shared memory, STAGES - 1
+// stages ahead.  A
+// token needs no reduction: every lane keeps its rows' share of the outputs of a whole stage, and the TOK * C shares
 // are then summed over the column's lanes so that each lane ends with some of the sums (fewer shuffles than sums).
-template <typename T, int RPT, int SPLIT, int C>
+template <typename T, int RPT, int SPLIT, int C, int TOK, int STAGES>
 __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs a) {
     pdl_sync();
     constexpr int DP = RPT * SPLIT;
     constexpr int COLS = DM_SCAN / SPLIT * C;
     constexpr int ROW = 4 * DP + 4;                     // a record
-    constexpr int NV = DM_TOK * C;
+    constexpr int NV = TOK * C;
     static_assert(NV % SPLIT == 0, "every lane ends with as many sums");
-    extern __shared__ __align__(16) float dm_sm[];      // [DM_STAGES][DM_TOK][ROW]
-    __shared__ __align__(8) unsigned long long bars[DM_STAGES];
+    extern __shared__ __align__(16) float dm_sm[];      // [STAGES][TOK][ROW]
+    __shared__ __align__(8) unsigned long long bars[STAGES];
     const int b = blockIdx.x, h = blockIdx.y;
     const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT * C;
     const int col0 = blockIdx.z * COLS, col = col0 + cl;
@@ -295,42 +293,42 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
     const float* rec = a.rec + (size_t)h * a.nt * ROW;
     const uint32_t bar0 = smem_u32(bars);
     if (tid == 0) {
-        for (int q = 0; q < DM_STAGES; ++q) mbar_init(bar0 + 8u * q, 1);
+        for (int q = 0; q < STAGES; ++q) mbar_init(bar0 + 8u * q, 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     __syncthreads();
-    const int stages = (t1 - t0 + DM_TOK - 1) / DM_TOK;
+    const int stages = (t1 - t0 + TOK - 1) / TOK;
     auto issue = [&](int q) {
-        const int ts = t0 + q * DM_TOK, n = min(DM_TOK, t1 - ts);
-        float* to = dm_sm + (size_t)(q % DM_STAGES) * (DM_TOK * ROW);
+        const int ts = t0 + q * TOK, n = min(TOK, t1 - ts);
+        float* to = dm_sm + (size_t)(q % STAGES) * (TOK * ROW);
         if (tid == 0) {
             const uint32_t bytes = (uint32_t)(n * ROW) * sizeof(float);
-            mbar_expect_tx(bar0 + 8u * (q % DM_STAGES), bytes);
-            bulk_load(smem_u32(to), rec + (size_t)ts * ROW, bytes, bar0 + 8u * (q % DM_STAGES));
+            mbar_expect_tx(bar0 + 8u * (q % STAGES), bytes);
+            bulk_load(smem_u32(to), rec + (size_t)ts * ROW, bytes, bar0 + 8u * (q % STAGES));
         }
         // tokens behind the last: nothing is written, nothing fades, nothing is read (so that a stage has no branches)
-        for (int idx = n * ROW + tid; idx < DM_TOK * ROW; idx += DM_SCAN) {
+        for (int idx = n * ROW + tid; idx < TOK * ROW; idx += DM_SCAN) {
             const int e = idx % ROW;
             to[idx] = e >= 2 * DP && e < 3 * DP ? 1.f : 0.f;
         }
     };
     int issued = 0;
-    for (; issued < DM_STAGES - 1 && issued < stages; ++issued) issue(issued);
+    for (; issued < STAGES - 1 && issued < stages; ++issued) issue(issued);
     for (int st = 0; st < stages; ++st) {
-        const bool ok = mbar_wait(bar0 + 8u * (st % DM_STAGES), (st / DM_STAGES) & 1, a.error, 31);
+        const bool ok = mbar_wait(bar0 + 8u * (st % STAGES), (st / STAGES) & 1, a.error, 31);
         // the stage has landed for everyone, and everyone is done with the stage before
         if (!__syncthreads_and(ok)) {
             if (tid == 0)
-                for (int q = st; q < issued; ++q) mbar_wait(bar0 + 8u * (q % DM_STAGES), (q / DM_STAGES) & 1, a.error, 32);
+                for (int q = st; q < issued; ++q) mbar_wait(bar0 + 8u * (q % STAGES), (q / STAGES) & 1, a.error, 32);
             return;
         }
         if (issued < stages) issue(issued++);
-        const int ts = t0 + st * DM_TOK;
-        const float* stage = dm_sm + (size_t)(st % DM_STAGES) * (DM_TOK * ROW);
-        const int n = min(DM_TOK, t1 - ts);
+        const int ts = t0 + st * TOK;
+        const float* stage = dm_sm + (size_t)(st % STAGES) * (TOK * ROW);
+        const int n = min(TOK, t1 - ts);
         float o[NV];
 #pragma unroll
-        for (int tt = 0; tt < DM_TOK; ++tt) {
+        for (int tt = 0; tt < TOK; ++tt) {
             const float* row = stage + tt * ROW;
             F2 v[C], d[C];
 #pragma unroll
@@ -395,21 +393,21 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
     }
 }
 
-template <typename T, int RPT, int SPLIT, int C>
+template <typename T, int RPT, int SPLIT, int C, int TOK, int STAGES>
 static int decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
     constexpr int COLS = DM_SCAN / SPLIT * C;
-    const size_t smem = (size_t)DM_STAGES * DM_TOK * (4 * RPT * SPLIT + 4) * sizeof(float);
+    const size_t smem = (size_t)STAGES * TOK * (4 * RPT * SPLIT + 4) * sizeof(float);
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
-        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(B, a.H, (a.dim + COLS - 1) / COLS);
     if (early)
-        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT, C>), grid, DM_SCAN, smem, s, a);
+        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>), grid, DM_SCAN, smem, s, a);
     else        // prompts: the blocks run for the whole sequence and want an SM each (see tb_launch_plain)
-        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT, C>, grid, dim3(DM_SCAN), smem, s, a);
+        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>, grid, dim3(DM_SCAN), smem, s, a);
     return tb_last_error();
 }
 
@@ -421,12 +419,19 @@ static int decay_scan_launch(DecayScanArgs a, int B, cudaStream_t s) {
     a.error = tc_error_ptr();
     if (!a.error) return tb_last_error();
     const bool early = a.nt <= 2 * B;
+    // Few sequences: small pieces of the state per thread, so that as many warps as there are keep the chain of a token
+    // short (16 heads of 128, one prompt of 2,048 tokens: 197 us with 4 rows of 2 columns, 245 with 8 of 2, 320 with 8
+    // of 4).  Enough of them to fill the GPU: larger pieces, which read a record's entry for more columns (eight
+    // prompts of 1,024 tokens: 444 us with 8 rows of 4 columns, 665 with 4 of 2).
+    const bool many = (long long)B * a.H * a.dim >= 128 * 32;
     switch (dm_rows(a.dim)) {
-        case 16: return decay_scan_go<T, 4, 4, 1>(a, B, early, s);
-        case 32: return decay_scan_go<T, 4, 8, 1>(a, B, early, s);
-        case 64: return decay_scan_go<T, 8, 8, 1>(a, B, early, s);
-        case 128: return decay_scan_go<T, 8, 16, 2>(a, B, early, s);
-        default: return decay_scan_go<T, 16, 16, 2>(a, B, early, s);
+        case 16: return decay_scan_go<T, 4, 4, 1, 8, 4>(a, B, early, s);
+        case 32: return decay_scan_go<T, 4, 8, 1, 8, 4>(a, B, early, s);
+        case 64:
+            return many ? decay_scan_go<T, 8, 8, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, 4, 16, 2, 16, 3>(a, B, early, s);
+        case 128:
+            return many ? decay_scan_go<T, 8, 16, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, 4, 32, 2, 16, 3>(a, B, early, s);
+        default: return decay_scan_go<T, 8, 32, 4, 8, 3>(a, B, early, s);
     }
 }
 
