@@ -2,6 +2,7 @@
 // heads of different sizes and a gate on the output: the general kernel (CUDA cores, float or bfloat16).
 //
 //   score(q at position p, key at position j) = cap(q . k * scale),   cap(s) = softcap * tanh(s / softcap)  (softcap > 0)
+//   a bias by distance (may be absent) is added to that: dist_bias[h][min(p - j, far)], far + 1 numbers a head
 //   visible iff j <= p and (p - j < window or j < keep_first) and (chunk == 0 or j / chunk == p / chunk)
 //   out[t, h, :] = softmax over the visible keys . v  * sigmoid(gate[t, h, :])                (gate may be absent)
 //   sink (may be absent): a number per head that joins the softmax's denominator as exp(sink_h), with no key and no
@@ -47,6 +48,8 @@ struct WinArgs {
     int gate_per_head = 0;  // 1: the gate holds one number per (token, head)
     float out_scale = 1.f;  // multiplies the output
     int ldo = 0;            // row pitch of out (0: nh * dv)
+    const float* dist_bias = nullptr;   // [nh, far + 1] or null
+    int far = 0;
 };
 
 template <typename T, int DPL>
@@ -127,6 +130,8 @@ __global__ void __launch_bounds__(AW_WARPS * 32) attention_window_kernel(const W
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s * inv_cap);
             const int j = key0 + lane;
+            if (a.dist_bias && j <= pos_r)
+                s += a.dist_bias[(size_t)(h0 + r % nheads) * (a.far + 1) + min(pos_r - j, a.far)];
             const bool see = j <= pos_r && (pos_r - j < a.window || j < a.keep_first) &&
                              (a.chunk <= 0 || j / a.chunk == pos_r / a.chunk);
             s = see ? s : -INFINITY;
@@ -267,6 +272,7 @@ static int window_launch(WinArgs a, int tiles, int nt, cudaStream_t s) {
     if (a.splits < 1 || (a.splits > 1 && !a.partial)) return TB_ERR_ARG;
     if (a.ldo == 0) a.ldo = a.nh * a.dv;
     if (a.ldo < a.nh * a.dv) return TB_ERR_ARG;
+    if (a.dist_bias && a.far < 0) return TB_ERR_ARG;
     if (a.chunk < 0 || (a.ocos && (!a.osin || a.dv % 2))) return TB_ERR_ARG;
     if (tiles <= 0 || nt <= 0) return tiles == 0 || nt == 0 ? 0 : TB_ERR_ARG;
     const int group = a.nh / a.nkvh;
@@ -318,6 +324,20 @@ extern "C" {
                   softcap, gate_per_head, out_scale, ldo};                                                            \
         return window_launch<T>(a, tiles, nt, s);                                                                     \
     }
+// The same with a bias by distance, [nh, far + 1] (and without the turning back of the output).
+#define TB_ATTENTION_WINDOW_BIASED(NAME, T)                                                                           \
+    int NAME(const void* q, void* out, const void* kc, const void* vc, const void* gate, const int* tile_seq,         \
+             const int* tile_t0, const int* tile_nq, const int* tok_pos, const int* page_table, float* partial,       \
+             int tiles, int nt, int max_pages, int q_stride, int gate_stride, int nh, int nkvh, int dk, int dv,       \
+             int splits, int window, int keep_first, float scale, float softcap, int chunk, const float* sinks,       \
+             int gate_per_head, float out_scale, int ldo, const float* dist_bias, int far, cudaStream_t s) {          \
+        WinArgs a{q, out, kc, vc, gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, nullptr,     \
+                  nullptr, chunk, max_pages, q_stride, gate_stride, nh, nkvh, dk, dv, 0, splits, window, keep_first,  \
+                  scale, softcap, gate_per_head, out_scale, ldo, dist_bias, far};                                     \
+        return window_launch<T>(a, tiles, nt, s);                                                                     \
+    }
+TB_ATTENTION_WINDOW_BIASED(tb_attention_window_biased_f32, float)
+TB_ATTENTION_WINDOW_BIASED(tb_attention_window_biased_bf16, __nv_bfloat16)
 TB_ATTENTION_WINDOW_HEADS(tb_attention_window_heads_f32, float)
 TB_ATTENTION_WINDOW_HEADS(tb_attention_window_heads_bf16, __nv_bfloat16)
 TB_ATTENTION_WINDOW(tb_attention_window_f32, float)
@@ -325,6 +345,8 @@ TB_ATTENTION_WINDOW(tb_attention_window_bf16, __nv_bfloat16)
 }
 
 #include "tape.h"
+TB_TAPE_REGISTER(tb_attention_window_biased_f32)
+TB_TAPE_REGISTER(tb_attention_window_biased_bf16)
 TB_TAPE_REGISTER(tb_attention_window_heads_f32)
 TB_TAPE_REGISTER(tb_attention_window_heads_bf16)
 TB_TAPE_REGISTER(tb_attention_window_f32)

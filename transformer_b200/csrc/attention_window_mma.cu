@@ -3,7 +3,9 @@
 // Same mathematics as the general windowed kernel (attention_window.cu):
 //   score = cap(q . k * scale), visible iff j <= p and (p - j < window or j < keep_first) and (no chunks or both in
 //   the same chunk), an optional sink per head in the denominator, an optional turning back of the output's pairs, softmax in float,
-//   out = softmax . v * sigmoid(gate); key heads of DK and value heads of DV entries.
+//   out = softmax . v * sigmoid(gate); key heads of DK and value heads of DV entries; an optional bias by distance,
+//   dist_bias[h][min(p - j, far)], is added to the (capped) score: pages that lie wholly beyond `far` take one number a
+//   row, the others read the table (a few KB, in L1).
 //
 // A block = one tile of query tokens of ONE sequence x ONE key/value head with ALL the query heads of its group:
 // row r of the block's 64 is (token r / group, head r % group), so a page of K and V that is brought to shared
@@ -46,11 +48,13 @@ struct WinMmaArgs {
     int gate_per_head = 0;  // 1: the gate holds one number per (token, head)
     float out_scale = 1.f;  // multiplies the output
     int ldo = 0;            // row pitch of out (0: nh * DV)
+    const float* dist_bias = nullptr;   // [nh, far + 1]
+    int far = 0;
 };
 
 __host__ __device__ constexpr int wm_blocks(int dk, int dv) { return (dk + dv) <= 256 ? 3 : 1; }
 
-template <int DK, int DV>
+template <int DK, int DV, bool BIAS>
 __global__ void __launch_bounds__(WM_THREADS, wm_blocks(DK, DV)) attention_window_mma_kernel(const WinMmaArgs a) {
     pdl_sync();
     constexpr int CHK = DK / 8, CHV = DV / 8;          // 16-byte chunks in a row of K / of V
@@ -125,6 +129,15 @@ __global__ void __launch_bounds__(WM_THREADS, wm_blocks(DK, DV)) attention_windo
     const uint32_t sq_addr = (uint32_t)__cvta_generic_to_shared(sq);
     const float LOG2E = 1.4426950408889634f;
     const float scale_l2 = a.scale * LOG2E, cap_l2 = a.softcap * LOG2E;
+    // BIAS: the rows' heads' biases
+    const float *bias_a = nullptr, *bias_b = nullptr;
+    float far_a = 0.f, far_b = 0.f;
+    if constexpr (BIAS) {
+        bias_a = a.dist_bias + (size_t)(g * group + row_a % group) * (a.far + 1);
+        bias_b = a.dist_bias + (size_t)(g * group + row_b % group) * (a.far + 1);
+        far_a = __ldg(bias_a + a.far) * LOG2E;
+        far_b = __ldg(bias_b + a.far) * LOG2E;
+    }
     const float pre_cap = a.softcap > 0.f ? a.scale / a.softcap * 2.0f * LOG2E : 0.f;
 
     for (int it = i_lo; it < i_hi; ++it) {
@@ -169,6 +182,7 @@ __global__ void __launch_bounds__(WM_THREADS, wm_blocks(DK, DV)) attention_windo
             const bool open = key0 + WM_KEYS - 1 <= pos_first &&
                               (pos_last - key0 < a.window || key0 + WM_KEYS - 1 < a.keep_first) &&
                               (a.chunk <= 0 || key0 / a.chunk == pos_last / a.chunk);
+            const bool all_far = !BIAS || pos_first - (key0 + WM_KEYS - 1) >= a.far;
             float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
             for (int nb = 0; nb < WM_KEYS / 8; ++nb) {
@@ -177,6 +191,14 @@ __global__ void __launch_bounds__(WM_THREADS, wm_blocks(DK, DV)) attention_windo
                     // score * log2 e, capped: cap tanh(y) = cap - 2 cap / (1 + e^{2y}), y = s * scale / cap
                     float v = a.softcap > 0.f ? cap_l2 - __fdividef(2.0f * cap_l2, 1.0f + exp2f(s[nb][c] * pre_cap))
                                               : s[nb][c] * scale_l2;
+                    if constexpr (BIAS) {
+                        if (all_far) {
+                            v += (c & 2) ? far_b : far_a;
+                        } else {
+                            const int back = ((c & 2) ? pos_b : pos_a) - (key0 + nb * 8 + tid4 * 2 + (c & 1));
+                            v += __ldg(((c & 2) ? bias_b : bias_a) + min(max(back, 0), a.far)) * LOG2E;
+                        }
+                    }
                     if (!open) {
                         const int key = key0 + nb * 8 + tid4 * 2 + (c & 1);
                         const int pos = (c & 2) ? pos_b : pos_a;
@@ -338,18 +360,18 @@ __global__ void attention_window_mma_merge_kernel(const float* __restrict__ part
     }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool BIAS>
 static int window_mma_launch(const WinMmaArgs& a, int nt, cudaStream_t s) {
     const size_t smem = ((size_t)(WM_ROWS + 2 * WM_KEYS) * ap_row(DK) + (size_t)WM_KEYS * ap_row(DV)) * sizeof(__nv_bfloat16);
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_window_mma_kernel<DK, DV>,
+        cudaError_t e = cudaFuncSetAttribute(attention_window_mma_kernel<DK, DV, BIAS>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(a.tiles, a.nkvh, a.splits);
-    TB_LAUNCH((attention_window_mma_kernel<DK, DV>), grid, WM_THREADS, smem, s, a);
+    TB_LAUNCH((attention_window_mma_kernel<DK, DV, BIAS>), grid, WM_THREADS, smem, s, a);
     int rc = tb_last_error();
     if (rc || a.splits == 1) return rc;
     dim3 mgrid(nt, a.nh);
@@ -370,7 +392,10 @@ static int window_mma_entry(WinMmaArgs a, int nt, int dk, int dv, cudaStream_t s
         return TB_ERR_UNSUPPORTED;
     if (!a.gate_per_head && (a.gate_stride % 8 || ((uintptr_t)a.gate & 15))) return TB_ERR_UNSUPPORTED;
     if (a.tiles == 0) return 0;
-#define WM_CASE(K, V) if (dk == K && dv == V) return window_mma_launch<K, V>(a, nt, s);
+    if (a.dist_bias && a.far < 0) return TB_ERR_ARG;
+#define WM_CASE(K, V)                                                       \
+    if (dk == K && dv == V)                                                 \
+        return a.dist_bias ? window_mma_launch<K, V, true>(a, nt, s) : window_mma_launch<K, V, false>(a, nt, s);
     WM_CASE(32, 32)
     WM_CASE(48, 48)
     WM_CASE(64, 64)
@@ -422,8 +447,24 @@ int tb_attention_window_mma_heads_bf16(const void* q, void* out, const void* kc,
                    softcap, gate_per_head, out_scale, ldo},
         nt, dk, dv, s);
 }
+// The same with a bias by distance, [nh, far + 1] (and without the turning back of the output).
+int tb_attention_window_mma_biased_bf16(const void* q, void* out, const void* kc, const void* vc, const void* gate,
+                                 const int* tile_seq, const int* tile_t0, const int* tile_nq, const int* tok_pos,
+                                 const int* page_table, float* partial, int tiles, int nt, int max_pages, int q_stride,
+                                 int gate_stride, int nh, int nkvh, int dk, int dv, int splits, int window,
+                                 int keep_first, float scale, float softcap, int chunk, const float* sinks,
+                                 int gate_per_head, float out_scale, int ldo, const float* dist_bias, int far,
+                                 cudaStream_t s) {
+    return window_mma_entry(
+        WinMmaArgs{(const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
+                   (const __nv_bfloat16*)gate, tile_seq, tile_t0, tile_nq, tok_pos, page_table, partial, sinks, nullptr,
+                   nullptr, chunk, tiles, max_pages, q_stride, gate_stride, nh, nkvh, splits, window, keep_first, scale,
+                   softcap, gate_per_head, out_scale, ldo, dist_bias, far},
+        nt, dk, dv, s);
+}
 }
 
 #include "tape.h"
 TB_TAPE_REGISTER(tb_attention_window_mma_bf16)
 TB_TAPE_REGISTER(tb_attention_window_mma_heads_bf16)
+TB_TAPE_REGISTER(tb_attention_window_mma_biased_bf16)

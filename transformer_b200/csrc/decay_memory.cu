@@ -17,17 +17,19 @@
 //   decay_scan_kernel   prompts: the recurrence token by token, a block = a sequence x a head x some columns of S, whose
 //                       rows are split over adjacent lanes, in registers; the lanes' sums meet only in the output, so
 //                       no token waits for another's reduction
+//                       (also the scan of a memory [dim, vdim] that is read after it is written to: csrc/gated_linear.cu)
 //   decay_step_kernel   one token per sequence: a block = a sequence x a head; decays, bonus, the state's way through the
 //                       registers, the head's norm and the gate in one kernel
 // Everything that enters the recurrence is float on both paths; x, r, k, v and the gate have the activations' type.
-#include "common.cuh"
+#include "memory_common.cuh"
 #include "tc_common.cuh"                // bulk copies, barriers with bounded waits
 
 constexpr int DM_MIXES = 5;             // r, k, v, gate, decay
 constexpr int DM_SCAN = 128;            // threads of a scan block
 
-__host__ __device__ inline int dm_rows(int dim) { return dim <= 16 ? 16 : dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
-__host__ __device__ inline int dm_record(int dim) { return 4 * dm_rows(dim) + 4; }
+// floats of a record's values (16-byte pieces), and of a record, r | k | w | v | bonus, 0, 0, 0
+__host__ __device__ inline int dm_values(int dim, int vdim) { return vdim == dim ? dm_rows(dim) : (vdim + 3) / 4 * 4; }
+__host__ __device__ inline int dm_record(int dim, int vdim) { return 3 * dm_rows(dim) + dm_values(dim, vdim) + 4; }
 __host__ __device__ inline long long dm_state(int H, int dim, int width) { return ((long long)H * dim * dim + width + 3) / 4 * 4; }
 
 // ---- the mixes ---------------------------------------------------------------------------------------------
@@ -110,52 +112,13 @@ static int shift_mix_launch(const void* x, const float* mu, const float* state, 
     return tb_last_error();
 }
 
-template <typename T, int V>
-__device__ __forceinline__ void dm_load(const T* p, float (&f)[V]) {
-    if constexpr (V == 1) {
-        f[0] = ldf(p);
-    } else if constexpr (sizeof(T) == 2) {
-        const uint2 raw = *reinterpret_cast<const uint2*>(p);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
-    } else {
-        const float4 a = *reinterpret_cast<const float4*>(p);
-        f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-    }
-}
-template <int V>
-__device__ __forceinline__ void dm_store(float* p, const float (&f)[V]) {
-    if constexpr (V == 1) *p = f[0];
-    else *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-}
-
 // ---- decays ------------------------------------------------------------------------------------------------
-// This lane's share of W2 row . ta: `parts` adjacent lanes take a row's pieces of eight (or entries) in turn.
-template <typename T>
-__device__ __forceinline__ float decay_dot(const T* __restrict__ w2row, const float* ta, int rank, int part, int parts) {
-    float acc = 0.f;
-    if ((rank & 7) == 0) {
-#pragma unroll 4
-        for (int q = part * 8; q < rank; q += parts * 8) {
-            float w[8];
-            load8(w2row + q, w);
-            const float4 t0 = *reinterpret_cast<const float4*>(ta + q);
-            const float4 t1 = *reinterpret_cast<const float4*>(ta + q + 4);
-            acc += w[0] * t0.x + w[1] * t0.y + w[2] * t0.z + w[3] * t0.w + w[4] * t1.x + w[5] * t1.y + w[6] * t1.z + w[7] * t1.w;
-        }
-        return acc;
-    }
-    for (int q = part; q < rank; q += parts) acc += ldf(w2row + q) * ta[q];
-    return acc;
-}
-
 // tanh of the decay's first projection, ready for the product with W2: in the activations' type a value is stored as the
 // sum of two (what its rounding leaves goes into the second half of the row, and the product's weight holds W2 twice), so
-// the product loses nothing that matters; in float it is stored as it is.
+// the product loses nothing that matters; in float it is stored as it is.  plain: the projection itself, without tanh.
 template <typename T>
 __global__ void __launch_bounds__(256) decay_tanh_kernel(const float* __restrict__ a, int lda, T* __restrict__ out, int nt,
-                                                         int rank, int ldo) {
+                                                         int rank, int ldo, int plain) {
     pdl_sync();
     const int n = nt * ldo;
     for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
@@ -164,7 +127,8 @@ __global__ void __launch_bounds__(256) decay_tanh_kernel(const float* __restrict
         const int e = q < half ? q : q - half;
         float v = 0.f;
         if (e < rank) {
-            v = tanhf(a[(size_t)t * lda + e]);
+            v = a[(size_t)t * lda + e];
+            if (!plain) v = tanhf(v);
             if (q >= half) {
                 T hi;
                 stf(&hi, v);
@@ -195,7 +159,7 @@ __global__ void __launch_bounds__(256) decay_prep_kernel(const DecayArgs p) {
     if (row >= p.nt * p.H) return;
     const int t = row / p.H, h = row - t * p.H, dim = p.dim, hd = p.H * dim;
     const int DP = dm_rows(dim);
-    float* rec = p.rec + ((size_t)h * p.nt + t) * dm_record(dim);
+    float* rec = p.rec + ((size_t)h * p.nt + t) * dm_record(dim, dim);
     const T* z = static_cast<const T*>(p.z) + (size_t)t * hd + h * dim;
     const size_t part = (size_t)p.nt * hd;
     float bonus = 0.f;
@@ -235,40 +199,26 @@ struct DecayScanArgs {
     float* state;           // [slots, pitch]
     int* error;             // set by a wait that runs out
     float* out;             // [nt, H dim]
-    const void* x;          // [nt, width]: a sequence's last row becomes its state's last input
+    const void* x;          // [nt, width]: a sequence's last row becomes its state's last input (null: there is none)
     const int* seq_start;
     const int* slots;
     long long pitch;
-    int nt, H, dim, width;
+    int nt, H, dim, width, vdim;
 };
-
-// two floats in one register pair, and the hardware's packed multiply-add on them
-union F2 {
-    float2 f;
-    unsigned long long u;
-};
-__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
-    F2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d.u) : "l"(a.u), "l"(b.u), "l"(c.u));
-    return d;
-}
-__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
-    F2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d.u) : "l"(a.u), "l"(b.u));
-    return d;
-}
 
 // RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): DM_SCAN / SPLIT * C columns a
 // block.  The records of TOK tokens at a time are one bulk copy to shared memory, STAGES - 1
 // stages ahead.  A
 // token needs no reduction: every lane keeps its rows' share of the outputs of a whole stage, and the TOK * C shares
 // are then summed over the column's lanes so that each lane ends with some of the sums (fewer shuffles than sums).
-template <typename T, int RPT, int SPLIT, int C, int TOK, int STAGES>
+// SQUARE: vdim equals dim (a record's length is then known when this is compiled).
+template <typename T, int RPT, int SPLIT, int C, int TOK, int STAGES, bool SQUARE>
 __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs a) {
     pdl_sync();
     constexpr int DP = RPT * SPLIT;
     constexpr int COLS = DM_SCAN / SPLIT * C;
-    constexpr int ROW = 4 * DP + 4;                     // a record
+    const int VP = SQUARE ? DP : dm_values(a.dim, a.vdim);
+    const int ROW = 3 * DP + VP + 4;                    // a record
     constexpr int NV = TOK * C;
     static_assert(NV % SPLIT == 0, "every lane ends with as many sums");
     extern __shared__ __align__(16) float dm_sm[];      // [STAGES][TOK][ROW]
@@ -276,19 +226,19 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
     const int b = blockIdx.x, h = blockIdx.y;
     const int tid = threadIdx.x, part = tid & (SPLIT - 1), cl = tid / SPLIT * C;
     const int col0 = blockIdx.z * COLS, col = col0 + cl;
-    const int dim = a.dim, H = a.H;
+    const int dim = a.dim, vdim = SQUARE ? dim : a.vdim, H = a.H;
     const int t0 = a.seq_start[b], t1 = a.seq_start[b + 1];
     if (t0 >= t1) return;
     float* slot = a.state + (size_t)a.slots[b] * a.pitch;
-    float* S = slot + (size_t)h * dim * dim;
+    float* S = slot + (size_t)h * dim * vdim;
     F2 s[C][RPT / 2];                                   // rows 2i, 2i + 1 of this lane's
 #pragma unroll
     for (int c = 0; c < C; ++c)
 #pragma unroll
         for (int i = 0; i < RPT / 2; ++i) {
             const int r = ((i >> 1) * SPLIT + part) * 4 + (i & 1) * 2;
-            s[c][i].f.x = (r < dim && col + c < dim) ? S[(size_t)r * dim + col + c] : 0.f;
-            s[c][i].f.y = (r + 1 < dim && col + c < dim) ? S[(size_t)(r + 1) * dim + col + c] : 0.f;
+            s[c][i].f.x = (r < dim && col + c < vdim) ? S[(size_t)r * vdim + col + c] : 0.f;
+            s[c][i].f.y = (r + 1 < dim && col + c < vdim) ? S[(size_t)(r + 1) * vdim + col + c] : 0.f;
         }
     const float* rec = a.rec + (size_t)h * a.nt * ROW;
     const uint32_t bar0 = smem_u32(bars);
@@ -333,7 +283,7 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
             F2 v[C], d[C];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                v[c].f.x = v[c].f.y = row[3 * DP + min(col + c, DP - 1)];
+                v[c].f.x = v[c].f.y = row[3 * DP + min(col + c, VP - 1)];
                 d[c].f.x = d[c].f.y = 0.f;
             }
 #pragma unroll
@@ -370,9 +320,9 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
 #pragma unroll
         for (int j = 0; j < NV / SPLIT; ++j) {
             const int idx = part * (NV / SPLIT) + j, tt = idx / C, c = idx % C;
-            if (tt < n && col + c < dim) {
+            if (tt < n && col + c < vdim) {
                 const float* row = stage + tt * ROW;
-                a.out[((size_t)(ts + tt) * H + h) * dim + col + c] = o[j] + row[4 * DP] * row[3 * DP + col + c];
+                a.out[((size_t)(ts + tt) * H + h) * vdim + col + c] = o[j] + row[3 * DP + VP] * row[3 * DP + col + c];
             }
         }
     }
@@ -381,39 +331,41 @@ __global__ void __launch_bounds__(DM_SCAN) decay_scan_kernel(const DecayScanArgs
 #pragma unroll
         for (int i = 0; i < RPT / 2; ++i) {
             const int r = ((i >> 1) * SPLIT + part) * 4 + (i & 1) * 2;
-            if (col + c < dim) {
-                if (r < dim) S[(size_t)r * dim + col + c] = s[c][i].f.x;
-                if (r + 1 < dim) S[(size_t)(r + 1) * dim + col + c] = s[c][i].f.y;
+            if (col + c < vdim) {
+                if (r < dim) S[(size_t)r * vdim + col + c] = s[c][i].f.x;
+                if (r + 1 < dim) S[(size_t)(r + 1) * vdim + col + c] = s[c][i].f.y;
             }
         }
-    if (h == 0 && blockIdx.z == 0) {        // the mixes have read the old one
+    if (h == 0 && blockIdx.z == 0 && a.x) {        // the mixes have read the old one
         const T* last = static_cast<const T*>(a.x) + (size_t)(t1 - 1) * a.width;
         float* to = slot + (size_t)H * dim * dim;
         for (int c = tid; c < a.width; c += DM_SCAN) to[c] = ldf(last + c);
     }
 }
 
-template <typename T, int RPT, int SPLIT, int C, int TOK, int STAGES>
+template <typename T, bool SQUARE, int RPT, int SPLIT, int C, int TOK, int STAGES>
 static int decay_scan_go(const DecayScanArgs& a, int B, bool early, cudaStream_t s) {
     constexpr int COLS = DM_SCAN / SPLIT * C;
-    const size_t smem = (size_t)STAGES * TOK * (4 * RPT * SPLIT + 4) * sizeof(float);
-    static bool configured = false;
-    if (smem > 48 * 1024 && !configured) {
-        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const size_t smem = (size_t)STAGES * TOK * dm_record(a.dim, a.vdim) * sizeof(float);
+    if (smem > 220 * 1024) return TB_ERR_UNSUPPORTED;
+    static size_t configured = 48 * 1024;
+    if (smem > configured) {
+        cudaError_t e = cudaFuncSetAttribute(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES, SQUARE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        configured = true;
+        configured = smem;
     }
-    dim3 grid(B, a.H, (a.dim + COLS - 1) / COLS);
+    dim3 grid(B, a.H, (a.vdim + COLS - 1) / COLS);
     if (early)
-        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>), grid, DM_SCAN, smem, s, a);
+        TB_LAUNCH((decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES, SQUARE>), grid, DM_SCAN, smem, s, a);
     else        // prompts: the blocks run for the whole sequence and want an SM each (see tb_launch_plain)
-        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES>, grid, dim3(DM_SCAN), smem, s, a);
+        tb_launch_plain(decay_scan_kernel<T, RPT, SPLIT, C, TOK, STAGES, SQUARE>, grid, dim3(DM_SCAN), smem, s, a);
     return tb_last_error();
 }
 
-template <typename T>
+template <typename T, bool SQUARE>
 static int decay_scan_launch(DecayScanArgs a, int B, cudaStream_t s) {
-    if (B < 0 || a.H <= 0 || a.dim <= 0 || a.width <= 0 || a.pitch < dm_state(a.H, a.dim, a.width)) return TB_ERR_ARG;
+    if (B < 0 || a.H <= 0 || a.dim <= 0 || a.vdim <= 0 || a.pitch < (long long)a.H * a.dim * a.vdim) return TB_ERR_ARG;
+    if (a.x && (a.width <= 0 || a.vdim != a.dim || a.pitch < dm_state(a.H, a.dim, a.width))) return TB_ERR_ARG;
     if (a.dim > 256) return TB_ERR_UNSUPPORTED;
     if (B == 0) return 0;
     a.error = tc_error_ptr();
@@ -423,15 +375,15 @@ static int decay_scan_launch(DecayScanArgs a, int B, cudaStream_t s) {
     // short (16 heads of 128, one prompt of 2,048 tokens: 197 us with 4 rows of 2 columns, 245 with 8 of 2, 320 with 8
     // of 4).  Enough of them to fill the GPU: larger pieces, which read a record's entry for more columns (eight
     // prompts of 1,024 tokens: 444 us with 8 rows of 4 columns, 665 with 4 of 2).
-    const bool many = (long long)B * a.H * a.dim >= 128 * 32;
+    const bool many = (long long)B * a.H * a.vdim >= 128 * 32;
     switch (dm_rows(a.dim)) {
-        case 16: return decay_scan_go<T, 4, 4, 1, 8, 4>(a, B, early, s);
-        case 32: return decay_scan_go<T, 4, 8, 1, 8, 4>(a, B, early, s);
+        case 16: return decay_scan_go<T, SQUARE, 4, 4, 1, 8, 4>(a, B, early, s);
+        case 32: return decay_scan_go<T, SQUARE, 4, 8, 1, 8, 4>(a, B, early, s);
         case 64:
-            return many ? decay_scan_go<T, 8, 8, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, 4, 16, 2, 16, 3>(a, B, early, s);
+            return many ? decay_scan_go<T, SQUARE, 8, 8, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, SQUARE, 4, 16, 2, 16, 3>(a, B, early, s);
         case 128:
-            return many ? decay_scan_go<T, 8, 16, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, 4, 32, 2, 16, 3>(a, B, early, s);
-        default: return decay_scan_go<T, 8, 32, 4, 8, 3>(a, B, early, s);
+            return many ? decay_scan_go<T, SQUARE, 8, 16, 4, 8, 4>(a, B, early, s) : decay_scan_go<T, SQUARE, 4, 32, 2, 16, 3>(a, B, early, s);
+        default: return decay_scan_go<T, SQUARE, 8, 32, 4, 8, 3>(a, B, early, s);
     }
 }
 
@@ -448,12 +400,12 @@ static int decay_prep_launch(const DecayArgs& p, cudaStream_t s) {
     return tb_last_error();
 }
 template <typename T>
-static int decay_tanh_launch(const float* a, int lda, void* out, int nt, int rank, int ldo, cudaStream_t s) {
+static int decay_tanh_launch(const float* a, int lda, void* out, int nt, int rank, int ldo, int plain, cudaStream_t s) {
     if (nt < 0 || rank <= 0 || lda < rank || ldo < rank * (sizeof(T) == 2 ? 2 : 1) || (sizeof(T) == 2 && ldo % 2)) return TB_ERR_ARG;
     if (nt == 0) return 0;
     const long long n = (long long)nt * ldo;
     if (n > (1ll << 30)) return TB_ERR_UNSUPPORTED;
-    TB_LAUNCH((decay_tanh_kernel<T>), (int)((n + 255) / 256 > 1184 ? 1184 : (n + 255) / 256), 256, 0, s, a, lda, (T*)out, nt, rank, ldo);
+    TB_LAUNCH((decay_tanh_kernel<T>), (int)((n + 255) / 256 > 1184 ? 1184 : (n + 255) / 256), 256, 0, s, a, lda, (T*)out, nt, rank, ldo, plain);
     return tb_last_error();
 }
 
@@ -602,7 +554,15 @@ static int decay_step_launch(const DecayStepArgs& p, int B, cudaStream_t s) {
 extern "C" {
 // Floats of state per slot.
 int tb_decay_state_size(int H, int dim, int width) { return (int)dm_state(H, dim, width); }
-int tb_decay_record_size(int dim) { return dm_record(dim); }
+int tb_decay_record_size(int dim) { return dm_record(dim, dim); }
+// The scan alone, of a memory [dim, vdim] per head that lies at the start of a slot's state; rec [H, nt, record size].
+int tb_decay_scan_rect_record_size(int dim, int vdim) { return dm_record(dim, vdim); }
+int tb_decay_scan_rect(const float* rec, float* state, long long pitch, float* out, const int* seq_start, const int* slots,
+                       int nt, int B, int H, int dim, int vdim, cudaStream_t s) {
+    if ((uintptr_t)rec & 15) return TB_ERR_ARG;
+    const DecayScanArgs a{rec, state, nullptr, out, nullptr, seq_start, slots, pitch, nt, H, dim, 0, vdim};
+    return vdim == dim ? decay_scan_launch<float, true>(a, B, s) : decay_scan_launch<float, false>(a, B, s);
+}
 // out [5, nt, d]: the mixes of every token; offsets [groups + 1] and row_group [groups nt] (may be null): the lists by
 // which one grouped product multiplies the first `groups` of them with a matrix each.  `at`: where in a slot's state the
 // last input lies.
@@ -614,7 +574,10 @@ int tb_decay_record_size(int dim) { return dm_record(dim); }
                                    slots, nt, d, s);                                                                  \
     }                                                                                                                 \
     int tb_decay_tanh_##SFX(const float* a, int lda, void* out, int nt, int rank, int ldo, cudaStream_t s) {          \
-        return decay_tanh_launch<T>(a, lda, out, nt, rank, ldo, s);                                                   \
+        return decay_tanh_launch<T>(a, lda, out, nt, rank, ldo, 0, s);                                                \
+    }                                                                                                                 \
+    int tb_split_rows_##SFX(const float* a, int lda, void* out, int nt, int rank, int ldo, cudaStream_t s) {          \
+        return decay_tanh_launch<T>(a, lda, out, nt, rank, ldo, 1, s);                                                \
     }                                                                                                                 \
     int tb_decay_prep_##SFX(const void* z, const float* pre, const float* w0, const float* u, float* rec,             \
                             int nt, int H, int dim, cudaStream_t s) {                                                 \
@@ -624,8 +587,9 @@ int tb_decay_record_size(int dim) { return dm_record(dim); }
     int tb_decay_scan_##SFX(const float* rec, float* state, long long pitch, float* out, const void* x, int width,    \
                             const int* seq_start, const int* slots, int nt, int B, int H, int dim, cudaStream_t s) {  \
         if ((uintptr_t)rec & 15) return TB_ERR_ARG;                                                                   \
-        return decay_scan_launch<T>(DecayScanArgs{rec, state, nullptr, out, x, seq_start, slots, pitch, nt, H, dim,   \
-                                                  width}, B, s);                                                      \
+        if (!x) return TB_ERR_ARG;                                                                                    \
+        return decay_scan_launch<T, true>(DecayScanArgs{rec, state, nullptr, out, x, seq_start, slots, pitch, nt, H,  \
+                                                        dim, width, dim}, B, s);                                      \
     }                                                                                                                 \
     int tb_decay_step_##SFX(const void* z, const void* x, int width, const float* a, int lda, const void* w2,         \
                             const float* w0, const float* u, const float* norm, float eps, float* state,              \
@@ -641,11 +605,14 @@ TB_DECAY(bf16, __nv_bfloat16)
 #include "tape.h"
 TB_TAPE_REGISTER(tb_shift_mix_f32)
 TB_TAPE_REGISTER(tb_shift_mix_bf16)
+TB_TAPE_REGISTER(tb_split_rows_f32)
+TB_TAPE_REGISTER(tb_split_rows_bf16)
 TB_TAPE_REGISTER(tb_decay_tanh_f32)
 TB_TAPE_REGISTER(tb_decay_tanh_bf16)
 TB_TAPE_REGISTER(tb_decay_prep_f32)
 TB_TAPE_REGISTER(tb_decay_prep_bf16)
 TB_TAPE_REGISTER(tb_decay_scan_f32)
 TB_TAPE_REGISTER(tb_decay_scan_bf16)
+TB_TAPE_REGISTER(tb_decay_scan_rect)
 TB_TAPE_REGISTER(tb_decay_step_f32)
 TB_TAPE_REGISTER(tb_decay_step_bf16)

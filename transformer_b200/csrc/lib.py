@@ -90,6 +90,19 @@ _SIGNATURES: Dict[str, str] = {
     "tb_decay_prep_f32": "pppppiii", "tb_decay_prep_bf16": "pppppiii",
     "tb_decay_scan_f32": "pplppippiiii", "tb_decay_scan_bf16": "pplppippiiii",
     "tb_decay_step_f32": "ppipippppfplpippiiiii", "tb_decay_step_bf16": "ppipippppfplpippiiiii",
+    "tb_qknorm_rope_cache_biased_f32": "pippppfpppippppiiiiiii", "tb_qknorm_rope_cache_biased_bf16": "pippppfpppippppiiiiiii",
+    "tb_attention_window_biased_f32": "pppppppppppiiiiiiiiiiiiffipifipi",
+    "tb_attention_window_biased_bf16": "pppppppppppiiiiiiiiiiiiffipifipi",
+    "tb_attention_window_mma_biased_bf16": "pppppppppppiiiiiiiiiiiiffipifipi",
+    "tb_split_rows_f32": "pipiii", "tb_split_rows_bf16": "pipiii",
+    "tb_decay_scan_rect": "pplpppiiiii",
+    "tb_gated_linear_prep_f32": "pipppiiiiiff", "tb_gated_linear_prep_bf16": "pipppiiiiiff",
+    "tb_gated_linear_step_f32": "pipipppplpippiiiiiifff", "tb_gated_linear_step_bf16": "pipipppplpippiiiiiifff",
+    "tb_split_delta_prep_f32": "pipippppiii", "tb_split_delta_prep_bf16": "pipippppiii",
+    "tb_split_delta_step_f32": "pipippppfplpippiiiii", "tb_split_delta_step_bf16": "pipippppfplpippiiiii",
+    "tb_split_delta_scan": "pplpppiiii",
+    "tb_stream_step_f32": "ppppipplpipppppii", "tb_stream_step_bf16": "ppppipplpipppppii",
+    "tb_embed_learned_f32": "pppppiifppp", "tb_embed_learned_bf16": "pppppiifppp",
     "tb_post_add_layernorm_router_f32": "pppppippfipppfipiippppiii",
     "tb_post_add_layernorm_router_bf16": "pppppippfipppfipiippppiii",
 }
@@ -112,7 +125,8 @@ class TapeMap(ctypes.Structure):
     _fields_ = [("base", ctypes.c_ulonglong), ("size", ctypes.c_ulonglong), ("delta", ctypes.c_longlong)]
 
 
-_NO_STREAM = {"tb_decay_state_size": "iii", "tb_decay_record_size": "i",
+_NO_STREAM = {"tb_decay_scan_rect_record_size": "ii", "tb_split_delta_record_size": "i",
+              "tb_decay_state_size": "iii", "tb_decay_record_size": "i",
               "tb_attention_window_mma_tile_tokens": "ii", "tb_delta_state_size": "iiiii", "tb_delta_record_size": "i", "tb_delta_scan_lanes": "i", "tb_delta_value_pitch": "i", "tb_mlstm_state_size": "ii", "tb_latent_attention_tile_tokens": "i", "tb_attention_tile_tokens": "ii", "tb_gemm_tc_status": "", "tb_attention_prefill_tile_tokens": "",
               "tb_attention_tc_tile_tokens": ""}
 
@@ -374,7 +388,8 @@ def kernel_status_async(host_int32: torch.Tensor) -> None:
 
 def _gave_up(code: int) -> str:
     """Which kernel family a wait code belongs to (1..5 tensor-core products, 11..17 tensor-core prompt
-    attention, 21..27 decode attention with the page ring, 31..32 the decaying memory's scan)."""
+    attention, 21..27 decode attention with the page ring, 31..32 the decaying memory's scan, 33..34 the split delta
+    rule's)."""
     if 1 <= code <= 5:
         return "tensor-core matrix product"
     if 11 <= code <= 17:
@@ -383,6 +398,8 @@ def _gave_up(code: int) -> str:
         return "decode attention"
     if 31 <= code <= 32:
         return "scan of the decaying memory"
+    if 33 <= code <= 34:
+        return "scan of the split delta rule"
     return "unknown kernel"
 
 
@@ -427,6 +444,16 @@ def decay_state_size(heads: int, dim: int, width: int) -> int:
 def decay_record_size(dim: int) -> int:
     """Floats of the record that the decaying memory's first kernel leaves the scan per (token, head)."""
     return library().tb_decay_record_size(dim)
+
+
+def gated_linear_record_size(dim: int, vdim: int) -> int:
+    """Floats of the record that the gated linear attention's first kernel leaves the scan per (token, head)."""
+    return library().tb_decay_scan_rect_record_size(dim, vdim)
+
+
+def split_delta_record_size(dim: int) -> int:
+    """Floats of the record that the split delta rule's first kernel leaves the scan per (token, head)."""
+    return library().tb_split_delta_record_size(dim)
 
 
 def attention_window_mma_tile_tokens(nh: int, nkvh: int) -> int:

@@ -178,8 +178,10 @@ static int rope_cache_launch(void* qkv, const int* tok_seq, const int* tok_pos, 
 
 // The same step for a mixer that norms its whole query and key projections first and rotates only a part of every
 // head, with value heads of a size of their own.  Row of z: q (nh dk) | k (nkvh dk) | v (nkvh dv) | ...
+//   bias [q | k | v] is added first (may be null);
 //   q <- q / sqrt(mean over ALL nh dk entries (q^2) + eps) * q_norm,   k alike over its nkvh dk entries;
 //   the first rdims entries of every head turn by the token's angles (table [positions, rdims / 2]), the rest pass;
+//   the queries are multiplied by q_mult[position] (may be null);
 //   q is written back in place, k and v go to the cache:  K [pages, nkvh, TB_PAGE, dk],  V [pages, nkvh, TB_PAGE, dv].
 // Statistics, the norm and the rotation are float; one rounding at each store.  A block per token.
 template <typename T>
@@ -188,18 +190,21 @@ qknorm_rope_cache_kernel(T* __restrict__ z, int ldz, const float* __restrict__ q
                          float eps, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                          const int* __restrict__ page_table, int max_pages, const float* __restrict__ cos_t,
                          const float* __restrict__ sin_t, T* __restrict__ kc, T* __restrict__ vc, int nh, int nkvh,
-                         int dk, int dv, int rdims, int half_pairing) {
+                         int dk, int dv, int rdims, int half_pairing, const float* __restrict__ bias,
+                         const float* __restrict__ q_mult) {
     pdl_sync();
     __shared__ float red[33];
     const int t = blockIdx.x;
     const int pos = tok_pos[t];
     const int nq = nh * dk, nk = nkvh * dk;
     T* row = z + (size_t)t * ldz;
+    auto entry = [&](int c) { return bias ? ldf(row + c) + bias[c] : ldf(row + c); };
+    const float qm = q_mult ? q_mult[pos] : 1.f;
     float rq = 1.f, rk = 1.f;
     if (q_norm) {
         float ss = 0.f;
         for (int c = threadIdx.x; c < nq; c += blockDim.x) {
-            const float x = ldf(row + c);
+            const float x = entry(c);
             ss += x * x;
         }
         rq = 1.0f / sqrtf(block_sum(ss, red) / (float)nq + eps);
@@ -207,7 +212,7 @@ qknorm_rope_cache_kernel(T* __restrict__ z, int ldz, const float* __restrict__ q
     if (k_norm) {
         float ss = 0.f;
         for (int c = threadIdx.x; c < nk; c += blockDim.x) {
-            const float x = ldf(row + nq + c);
+            const float x = entry(nq + c);
             ss += x * x;
         }
         rk = 1.0f / sqrtf(block_sum(ss, red) / (float)nk + eps);
@@ -228,9 +233,9 @@ qknorm_rope_cache_kernel(T* __restrict__ z, int ldz, const float* __restrict__ q
         const int base = head * dk;             // column of the head's first entry in the row (q and k are adjacent)
         const float* w = is_q ? q_norm : k_norm;
         const int wb = is_q ? base : base - nq;
-        const float r = is_q ? rq : rk;
-        const float x0 = ldf(row + base + i0) * r * (w ? w[wb + i0] : 1.f);
-        const float x1 = ldf(row + base + i1) * r * (w ? w[wb + i1] : 1.f);
+        const float r = is_q ? rq * qm : rk;
+        const float x0 = entry(base + i0) * r * (w ? w[wb + i0] : 1.f);
+        const float x1 = entry(base + i1) * r * (w ? w[wb + i1] : 1.f);
         const float c = cs[i], s = sn[i];
         const float y0 = x0 * c - x1 * s, y1 = x1 * c + x0 * s;
         if (is_q) {
@@ -249,14 +254,14 @@ qknorm_rope_cache_kernel(T* __restrict__ z, int ldz, const float* __restrict__ q
         const bool is_q = head < nh;
         const int base = head * dk;
         const float* w = is_q ? q_norm : k_norm;
-        const float y = ldf(row + base + c) * (is_q ? rq : rk) * (w ? w[(is_q ? base : base - nq) + c] : 1.f);
+        const float y = entry(base + c) * (is_q ? rq * qm : rk) * (w ? w[(is_q ? base : base - nq) + c] : 1.f);
         if (is_q) stf(row + base + c, y);
         else if (kc) stf(kc + (cache_row + (size_t)(head - nh) * TB_PAGE) * dk + c, y);
     }
     if (vc)
         for (int idx = threadIdx.x; idx < nkvh * dv; idx += blockDim.x) {
             const int head = idx / dv, c = idx - head * dv;
-            vc[(cache_row + (size_t)head * TB_PAGE) * dv + c] = row[nq + nk + idx];
+            stf(vc + (cache_row + (size_t)head * TB_PAGE) * dv + c, entry(nq + nk + idx));
         }
 }
 
@@ -268,19 +273,29 @@ qknorm_rope_cache_vec_kernel(T* __restrict__ z, int ldz, const float* __restrict
                              const float* __restrict__ k_norm, float eps, const int* __restrict__ tok_seq,
                              const int* __restrict__ tok_pos, const int* __restrict__ page_table, int max_pages,
                              const float* __restrict__ cos_t, const float* __restrict__ sin_t, T* __restrict__ kc,
-                             T* __restrict__ vc, int nh, int nkvh, int dk, int dv, int rdims) {
+                             T* __restrict__ vc, int nh, int nkvh, int dk, int dv, int rdims,
+                             const float* __restrict__ bias, const float* __restrict__ q_mult) {
     pdl_sync();
     __shared__ float red[33];
     const int t = blockIdx.x;
     const int pos = tok_pos[t];
     const int nq = nh * dk, nk = nkvh * dk;
     T* row = z + (size_t)t * ldz;
+    auto entries = [&](int c, float (&x)[8]) {
+        load8(row + c, x);
+        if (!bias) return;
+        float b[8];
+        load8(bias + c, b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += b[e];
+    };
+    const float qm = q_mult ? q_mult[pos] : 1.f;
     float rq = 1.f, rk = 1.f;
     if (q_norm) {
         float ss = 0.f;
         for (int c = threadIdx.x * 8; c < nq; c += blockDim.x * 8) {
             float x[8];
-            load8(row + c, x);
+            entries(c, x);
 #pragma unroll
             for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
         }
@@ -290,7 +305,7 @@ qknorm_rope_cache_vec_kernel(T* __restrict__ z, int ldz, const float* __restrict
         float ss = 0.f;
         for (int c = threadIdx.x * 8; c < nk; c += blockDim.x * 8) {
             float x[8];
-            load8(row + nq + c, x);
+            entries(nq + c, x);
 #pragma unroll
             for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
         }
@@ -310,12 +325,16 @@ qknorm_rope_cache_vec_kernel(T* __restrict__ z, int ldz, const float* __restrict
         const float* w = is_q ? q_norm : k_norm;
         const float r = is_q ? rq : rk;
         float x[8], y[8];
-        load8(row + c, x);
+        entries(c, x);
         if (w) {
             float wv[8];
             load8(w + (is_q ? c : c - nq), wv);
 #pragma unroll
             for (int e = 0; e < 8; ++e) x[e] *= r * wv[e];
+        }
+        if (is_q && q_mult) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) x[e] *= qm;
         }
         if (within < rdims) {           // four pairs, angles within / 2 .. within / 2 + 3
             const float4 c4 = *reinterpret_cast<const float4*>(cs + (within >> 1));
@@ -337,7 +356,7 @@ qknorm_rope_cache_vec_kernel(T* __restrict__ z, int ldz, const float* __restrict
         for (int c = threadIdx.x * 8; c < nkvh * dv; c += blockDim.x * 8) {
             const int head = c / dv, within = c - head * dv;
             float x[8];
-            load8(row + nq + nk + c, x);
+            entries(nq + nk + c, x);
             store8(vc + (cache_row + (size_t)head * TB_PAGE) * dv + within, x);
         }
 }
@@ -346,19 +365,20 @@ template <typename T>
 static int qknorm_rope_cache_launch(void* z, int ldz, const float* q_norm, const float* k_norm, float eps,
                                     const int* tok_seq, const int* tok_pos, const int* page_table, int max_pages,
                                     const float* cos_t, const float* sin_t, void* kc, void* vc, int nt, int nh,
-                                    int nkvh, int dk, int dv, int rdims, int half_pairing, cudaStream_t s) {
+                                    int nkvh, int dk, int dv, int rdims, int half_pairing, const float* bias,
+                                    const float* q_mult, cudaStream_t s) {
     if (nt < 0 || nh <= 0 || nkvh <= 0 || dk <= 0 || dv <= 0 || rdims < 0 || rdims > dk || (rdims & 1)) return TB_ERR_ARG;
     if ((kc == nullptr) != (vc == nullptr) || ldz < (nh + nkvh) * dk + nkvh * dv) return TB_ERR_ARG;
     if (nt == 0) return 0;
     if (!half_pairing && dk % 8 == 0 && dv % 8 == 0 && rdims % 8 == 0 && ldz % 8 == 0 &&
         (((uintptr_t)z | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)q_norm | (uintptr_t)k_norm | (uintptr_t)cos_t |
-          (uintptr_t)sin_t) & 15) == 0) {
+          (uintptr_t)sin_t | (uintptr_t)bias) & 15) == 0) {
         TB_LAUNCH((qknorm_rope_cache_vec_kernel<T>), nt, 256, 0, s, (T*)z, ldz, q_norm, k_norm, eps, tok_seq, tok_pos,
-                  page_table, max_pages, cos_t, sin_t, (T*)kc, (T*)vc, nh, nkvh, dk, dv, rdims);
+                  page_table, max_pages, cos_t, sin_t, (T*)kc, (T*)vc, nh, nkvh, dk, dv, rdims, bias, q_mult);
         return tb_last_error();
     }
     TB_LAUNCH((qknorm_rope_cache_kernel<T>), nt, 256, 0, s, (T*)z, ldz, q_norm, k_norm, eps, tok_seq, tok_pos, page_table,
-              max_pages, cos_t, sin_t, (T*)kc, (T*)vc, nh, nkvh, dk, dv, rdims, half_pairing);
+              max_pages, cos_t, sin_t, (T*)kc, (T*)vc, nh, nkvh, dk, dv, rdims, half_pairing, bias, q_mult);
     return tb_last_error();
 }
 
@@ -381,8 +401,21 @@ int tb_rope_cache_bf16(void* qkv, const int* tok_seq, const int* tok_pos, const 
              void* kc, void* vc, int nt, int nh, int nkvh, int dk, int dv, int rdims, int half_pairing,               \
              cudaStream_t s) {                                                                                        \
         return qknorm_rope_cache_launch<T>(z, ldz, q_norm, k_norm, eps, tok_seq, tok_pos, page_table, max_pages,      \
-                                           cos_t, sin_t, kc, vc, nt, nh, nkvh, dk, dv, rdims, half_pairing, s);       \
+                                           cos_t, sin_t, kc, vc, nt, nh, nkvh, dk, dv, rdims, half_pairing, nullptr,  \
+                                           nullptr, s);                                                               \
     }
+// The same with a bias on the projections, [nh dk | nkvh dk | nkvh dv], and a multiplier of the queries by position.
+#define TB_QKNORM_ROPE_BIASED(NAME, T)                                                                                 \
+    int NAME(void* z, int ldz, const float* bias, const float* q_mult, const float* q_norm, const float* k_norm,      \
+             float eps, const int* tok_seq, const int* tok_pos, const int* page_table, int max_pages,                 \
+             const float* cos_t, const float* sin_t, void* kc, void* vc, int nt, int nh, int nkvh, int dk, int dv,    \
+             int rdims, int half_pairing, cudaStream_t s) {                                                           \
+        return qknorm_rope_cache_launch<T>(z, ldz, q_norm, k_norm, eps, tok_seq, tok_pos, page_table, max_pages,      \
+                                           cos_t, sin_t, kc, vc, nt, nh, nkvh, dk, dv, rdims, half_pairing, bias,     \
+                                           q_mult, s);                                                                \
+    }
+TB_QKNORM_ROPE_BIASED(tb_qknorm_rope_cache_biased_f32, float)
+TB_QKNORM_ROPE_BIASED(tb_qknorm_rope_cache_biased_bf16, __nv_bfloat16)
 TB_QKNORM_ROPE(tb_qknorm_rope_cache_f32, float)
 TB_QKNORM_ROPE(tb_qknorm_rope_cache_bf16, __nv_bfloat16)
 }
@@ -393,3 +426,5 @@ TB_TAPE_REGISTER(tb_rope_cache_f32)
 TB_TAPE_REGISTER(tb_rope_cache_bf16)
 TB_TAPE_REGISTER(tb_qknorm_rope_cache_f32)
 TB_TAPE_REGISTER(tb_qknorm_rope_cache_bf16)
+TB_TAPE_REGISTER(tb_qknorm_rope_cache_biased_f32)
+TB_TAPE_REGISTER(tb_qknorm_rope_cache_biased_bf16)

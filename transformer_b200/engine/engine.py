@@ -20,8 +20,8 @@ import torch
 from ..cache.paged import Cache
 from ..cache.slots import CacheError
 from ..csrc import lib
-from ..parts.block import build_layer, resolve
-from ..parts.base import EMBEDDINGS, HEADS, JOINTS, NORMS, NormedDelta, PairDelta, StreamRows
+from ..parts.block import add_pending, build_layer, resolve
+from ..parts.base import EMBEDDINGS, HEADS, JOINTS, NORMS, DepthSum, GatedDelta, NormedDelta, PairDelta, StreamRows
 from ..parts.spec import ModelSpec
 from .context import StepContext, Workspace, weak_callback
 from .tape import LayerTape, moves, run_tensors
@@ -42,6 +42,11 @@ def _pending_signature(pending):
         return ("s", pending.rows.data_ptr(), tuple(pending.rows.shape))
     if isinstance(pending, PairDelta):
         return ("p", _pending_signature(pending.first), _pending_signature(pending.second))
+    if isinstance(pending, GatedDelta):       # names weights of the layer before: equal only for the same layer
+        return ("g",) + tuple(_pending_signature(t) for t in (pending.delta, pending.delta_bias, pending.gate, pending.gate_bias))
+    if isinstance(pending, DepthSum):
+        return ("d", _pending_signature(pending.pending), _pending_signature(pending.history),
+                _pending_signature(pending.weights), pending.terms)
     if isinstance(pending, NormedDelta):      # names a weight of the layer before: equal only for the same layer
         return ("n", _pending_signature(pending.delta), pending.weight.data_ptr(), pending.eps,
                 0 if pending.bias is None else pending.bias.data_ptr(), pending.center)
@@ -363,6 +368,11 @@ class Engine:
             if entry.joint is not None:
                 pending = self.joints[entry.joint].forward(ctx, x, pending)
             kind = self._run_kind[r] if taping else None
+            if kind is not None and isinstance(pending, DepthSum) and not ctx.decode:
+                # many tokens: the sum is done here, so that the layer's launches name no tensor of the joint's (layers
+                # of equal parts are then replayed with their own tensors put in)
+                add_pending(ctx, x, pending)
+                pending = None
             if kind is None:
                 pending = layer.forward(ctx, x, pending, self.cache.view(r), self.cache.state_of(r))
                 continue
@@ -383,6 +393,8 @@ class Engine:
                 pending = layer.forward(ctx, x, pending, self.cache.view(r), self.cache.state_of(r))
             else:
                 pending = tape.replay(maps[0], maps[1], self._run_tensors[r])
+        if self.spec.last_joint is not None:
+            pending = self.joints[self.spec.last_joint].forward(ctx, x, pending)
         n_out = len(ctx.h_want)
         logits = logits_out if logits_out is not None else \
             torch.empty((n_out, V), dtype=torch.float32, device=self.device)

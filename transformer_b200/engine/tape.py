@@ -21,6 +21,7 @@ from typing import List, Optional, Sequence
 import torch
 
 from ..csrc import lib
+from ..parts.base import GatedDelta
 
 
 class LayerTape:
@@ -61,6 +62,7 @@ class LayerTape:
         if calls:
             segments.append(("launches", lib.tape_entries(calls)))
         self._segments = segments
+        self._where = where
 
     def replay(self, maps, n_maps: int, tensors: Sequence[torch.Tensor]):
         for seg in self._segments:
@@ -69,6 +71,8 @@ class LayerTape:
             else:
                 _, a, at, out = seg
                 torch.mm(a, tensors[at].t(), out=out)
+        if isinstance(self.result, GatedDelta):      # it names weights of the recorded run's layer
+            return self.result.moved(lambda t: t if t is None else tensors[self._where[t.data_ptr()]])
         return self.result
 
 

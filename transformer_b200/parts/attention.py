@@ -13,6 +13,12 @@ the WHOLE query projection and the whole key projection before the rotation (``q
 below the head's); a gate on the output, o * sigmoid(Wg x1), whose projection rides in the merged product
 (``gate``).  With any of them the step runs  merged product -> norm + rotation + cache write (one kernel) ->
 windowed attention with the gate in its epilogue -> output product  (csrc/attention_window.cu, rope_cache.cu).
+To the same family belong: biases on the query, key and value projections (``bias``, weights ``bqkv``); a multiplier of
+the queries that grows with the position, 1 + coef ln(floor((p + 1) / every) + 1) (``query_temp`` = (coef, every), for
+``positions`` positions); a learned bias that is added to the score of a key n positions back, one number per
+(bucket of n, head) (``distance_bias`` = (rows, far), weights ``rel``; :func:`distance_bucket`); a multiplier of the
+output (``out_scale``); a bias on the output projection, which the block adds (``out_bias``, weights ``bo``).  Attention
+of this family can leave its heads' outputs in a wider row (``forward_rows``).
 
 A second family, again parameters of the same mixer: a short causal convolution over time on every channel of the
 q, k and v projections, ``conv_taps`` wide (weights ``conv``; the last ``conv_taps - 1`` projected rows are state of
@@ -55,6 +61,26 @@ USE_DECODE_RING = True  # decoding: the kernel with a ring of cache pages (TMA, 
 FUSE_DECODE_ROPE = True # decoding: that kernel also rotates q and k and writes the cache (no rotary kernel)
 RING_BLOCKS_PER_SM = 2  # decoding: the keys are sliced until that kernel has this many blocks per SM
 USE_WINDOW_MMA = True   # the windowed path, bfloat16: the tensor-core kernel before the general one
+
+
+def distance_bucket(n: int, rows: int, far: int) -> int:
+    """The row of a distance bias table with ``rows`` rows for a key ``n`` positions back: one row for each of the first
+    rows // 2 distances, then rows that widen with the logarithm of the distance, the last of them from ``far`` on at
+    the latest."""
+    half = rows // 2
+    if n < half:
+        return n
+    # a hair is added so that a quotient that is a whole number does not fall below it by rounding
+    steps = math.floor(math.log(n / half) / math.log(far / half) * (rows - half) + 1e-9)
+    return min(rows - 1, half + steps)
+
+
+def distance_buckets(rows: int, far: int):
+    """The buckets of the distances 0, 1, ... up to the first that has the last row (all further ones have it too)."""
+    out = [0]
+    while out[-1] < rows - 1:
+        out.append(distance_bucket(len(out), rows, far))
+    return out
 
 
 @MIXERS.register("attention")
@@ -101,22 +127,31 @@ class Attention(Mixer):
         self.head_gate = bool(params.get("head_gate", False))
         self.out_scale = float(params.get("out_scale", 1.0))
         self.sink_value = params.get("sink_value")
-        if not self.keyed and (self.bias or self.head_gate or self.out_scale != 1.0 or self.sink_value is not None or
-                               self.qk_norm == "unit"):
-            raise ValueError("biases, a gate per head, a fixed sink, an output multiplier and a norm without weights go "
-                             "with values that are the keys")
+        if not self.keyed and (self.head_gate or self.sink_value is not None or self.qk_norm == "unit"):
+            raise ValueError("a gate per head, a fixed sink and a norm without weights go with values that are the keys")
+        self.query_temp = params.get("query_temp")              # (coef, every)
+        self.distance_bias = params.get("distance_bias")        # (rows, far)
+        self.has_out_bias = bool(params.get("out_bias", False))
+        if self.query_temp is not None and not (float(self.query_temp[1]) > 0 and int(params.get("positions") or 0) > 0):
+            raise ValueError("a query multiplier by position needs a positive interval and the number of positions")
+        if self.distance_bias is not None and not (self.distance_bias[0] >= 2 and self.distance_bias[1] > self.distance_bias[0] // 2):
+            raise ValueError(f"a bias by distance needs two rows and a far distance above half of them, got {self.distance_bias}")
+        biased = bool(self.bias or self.out_scale != 1.0 or self.has_out_bias or self.query_temp or self.distance_bias)
+        if self.keyed and (self.has_out_bias or self.query_temp or self.distance_bias):
+            raise ValueError("an output bias, a query multiplier by position and a bias by distance go with values of their own")
         # the second family of mechanisms: its own kernel between the product and the attention
         self.prepared = bool(self.conv_taps or self.qk_norm == "head" or self.temperature or self.value_rotation or
                              self.value_mix)
-        if self.prepared and (self.gate or self.qk_norm == "whole"):
-            raise ValueError("a norm over the whole projection or an output gate does not go with the per-head family")
+        if self.prepared and (self.gate or self.qk_norm == "whole" or biased):
+            raise ValueError("a norm over the whole projection, an output gate, biases, an output multiplier and a query "
+                             "multiplier by position do not go with the per-head family")
         if self.keyed and (self.prepared or self.gate or self.sink or self.qk_norm == "whole" or self.dv != self.dh):
             raise ValueError("values that are the keys go with the parameters of their own family, a window, a chunk and a cap")
         if self.dv <= 0 or self.dv > 256 or self.window < 0 or self.keep_first < 0 or self.softcap < 0:
             raise ValueError("value heads of 1..256 entries; window, keep_first and softcap not negative")
         # any of the further mechanisms takes the step to the windowed kernels
         self.extended = bool(self.dv != self.dh or self.softcap or self.window or self.qk_norm or self.gate or
-                             "scale" in params or self.prepared or self.chunk or self.sink or self.keyed)
+                             "scale" in params or self.prepared or self.chunk or self.sink or self.keyed or biased)
         if not self.extended and (self.dh % 16):
             raise ValueError(f"the attention kernels take head sizes 16, 32, ..., 256; got {self.dh}")
         self.rdims = 0
@@ -139,7 +174,13 @@ class Attention(Mixer):
         if self.keyed:      # q | k | one gate per head; the bound weight gets rows of zeros up to a multiple of eight
             self.proj_rows = (self.nh + self.nkvh) * self.dh + (self.nh if self.head_gate else 0)
             self.qkv_width = (self.proj_rows + 7) // 8 * 8
-            self.rows_width = self.nh * self.dh
+        if self.extended and not self.prepared:
+            self.rows_width = self.nh * self.dv
+        self.q_mult = None
+        if self.query_temp is not None:
+            coef, every = float(self.query_temp[0]), int(self.query_temp[1])
+            self.q_mult = torch.tensor([1.0 + coef * math.log((p + 1) // every + 1.0) for p in range(int(params["positions"]))],
+                                       dtype=torch.float32, device=device)
         self.scale = float(params["scale"]) if "scale" in params else 1.0 / math.sqrt(self.dh)
         # query tiles this mixer asks the step to plan: the general kernel's, and the prompt kernel's
         self.general_tile = lib.attention_tile_tokens(self.nh, self.nkvh)
@@ -172,8 +213,14 @@ class Attention(Mixer):
         elif self.qk_norm == "head":
             decl["q_norm"] = ParamDecl((self.dh,), "norm", "ones")
             decl["k_norm"] = ParamDecl((self.dh,), "norm", "ones")
-        if self.bias:
+        if self.bias and self.keyed:
             decl["bqk"] = ParamDecl(((self.nh + self.nkvh) * self.dh,), "norm", "normal")
+        elif self.bias:
+            decl["bqkv"] = ParamDecl(((self.nh + self.nkvh) * self.dh + self.nkvh * self.dv,), "norm", "normal")
+        if self.distance_bias is not None:
+            decl["rel"] = ParamDecl((int(self.distance_bias[0]), self.nh), "norm", "normal")
+        if self.has_out_bias:
+            decl["bo"] = ParamDecl((self.d,), "norm", "normal")
         if self.conv_taps:
             decl["conv"] = ParamDecl((self.qkv_width, self.conv_taps), "norm", "normal")
         if self.temperature:
@@ -196,6 +243,12 @@ class Attention(Mixer):
                 self.weights["wqkv"] = torch.cat([w, w.new_zeros((self.qkv_width - self.proj_rows, self.d))]).contiguous()
             if self.sink_value is not None:
                 self.weights["sink"] = torch.full((self.nh,), float(self.sink_value), dtype=torch.float32, device=w.device)
+        if self.distance_bias is not None:      # the table by distance instead of by bucket, a head's numbers in a row
+            at = torch.tensor(distance_buckets(*(int(v) for v in self.distance_bias)), device=self.weights["rel"].device)
+            self.weights["rel"] = self.weights["rel"].float()[at].t().contiguous()
+        if self.has_out_bias:
+            self.weights["bo"] = (self.weights["bo"].float() * self.out_scale).contiguous()
+            self.out_bias = self.weights["bo"]
         if "vmix" in self.weights:
             self.weights["vmix"] = self.weights["vmix"].float().reshape(1).contiguous()
         if self.prepared and self.rdims and self.position.rotation()[2]:
@@ -258,8 +311,8 @@ class Attention(Mixer):
                              sinks=w.get("sink"), ocos=vcos, osin=vsin)
         matmul_nt(o, w["wo"], out)
 
-    def _forward_window(self, ctx, x1, out, cache) -> None:
-        """The step with the further mechanisms: see the head of this file."""
+    def _window_rows(self, ctx, x1, rows, cache) -> None:
+        """The step with the further mechanisms up to its output product: see the head of this file."""
         nt = x1.shape[0]
         sfx = lib.suffix(self.dtype)
         w = self.weights
@@ -271,21 +324,26 @@ class Attention(Mixer):
         if self.rdims:
             cos, sin, half = self.position.rotation()
         kc, vc = (cache.k, cache.v) if cache.writable else (None, None)
-        lib.call("tb_qknorm_rope_cache_" + sfx, lib.ptr(z), self.qkv_width, lib.ptr(w.get("q_norm")),
+        which, first = "", ()
+        if self.bias or self.q_mult is not None:
+            which, first = "biased_", (lib.ptr(w.get("bqkv")), lib.ptr(self.q_mult))
+        lib.call("tb_qknorm_rope_cache_" + which + sfx, lib.ptr(z), self.qkv_width, *first, lib.ptr(w.get("q_norm")),
                  lib.ptr(w.get("k_norm")), self.eps, lib.ptr(ctx.tok_seq), lib.ptr(ctx.tok_pos), lib.ptr(table),
                  ctx.max_pages, lib.ptr(cos), lib.ptr(sin), lib.ptr(kc), lib.ptr(vc), nt, self.nh, self.nkvh, self.dh,
                  self.dv, self.rdims, half)
-        o = ctx.scratch("attn.o", (nt, self.nh * self.dv), self.dtype)
         gate = z[:, (self.nh + self.nkvh) * self.dh + self.nkvh * self.dv:] if self.gate else None
         window = self.window if self.window else 1 << 30
-        run_window_attention(ctx, self, z, o, gate, cache, table, nt, window,
-                             sinks=w.get("sink") if self.sink else None)
-        matmul_nt(o, w["wo"], out)
+        plain = self.out_scale == 1.0 and rows.stride(0) == self.nh * self.dv
+        run_window_attention(ctx, self, z, rows, gate, cache, table, nt, window, sinks=w.get("sink") if self.sink else None,
+                             heads=None if plain else (0, self.out_scale, rows.stride(0)), dist_bias=w.get("rel"))
 
     def forward_rows(self, ctx, x1, rows, cache, state) -> None:
-        """The heads' outputs, gated and scaled, for the family whose values are the keys."""
+        """The heads' outputs, gated and scaled."""
+        if self.rows_width is None:
+            raise NotImplementedError("attention of this family does not leave its rows to another part's product")
         if not self.keyed:
-            raise NotImplementedError("only attention whose values are the keys leaves its rows to another part's product")
+            self._window_rows(ctx, x1, rows, cache)
+            return
         nt = x1.shape[0]
         w = self.weights
         z = ctx.scratch("attn.qkv", (nt, self.qkv_width), self.dtype)        # q | k | gate per head | padding
@@ -306,16 +364,13 @@ class Attention(Mixer):
                              heads=(1 if self.head_gate else 0, self.out_scale, rows.stride(0)))
 
     def forward(self, ctx, x1, out, cache, state) -> None:
-        if self.keyed:
+        if self.rows_width is not None:
             rows = ctx.scratch("attn.o", (x1.shape[0], self.rows_width), self.dtype)
             self.forward_rows(ctx, x1, rows, cache, state)
             matmul_nt(rows, self.weights["wo"], out)
             return
         if self.prepared:
             self._forward_prepared(ctx, x1, out, cache, state)
-            return
-        if self.extended:
-            self._forward_window(ctx, x1, out, cache)
             return
         nt = x1.shape[0]
         sfx = lib.suffix(self.dtype)
@@ -419,11 +474,16 @@ class Attention(Mixer):
 
 
 def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=None, sinks=None, ocos=None,
-                         osin=None, heads=None) -> None:
+                         osin=None, heads=None, dist_bias=None) -> None:
     """The windowed attention of the step's rotated queries ``z`` over the cache, into ``o`` (gate applied).
     ``sinks``: a number per head in the softmax's denominator; ``ocos, osin``: tables that turn the output back;
-    ``heads`` = (gate holds one number per head, output multiplier, pitch of ``o``)."""
+    ``heads`` = (gate holds one number per head, output multiplier, pitch of ``o``); ``dist_bias``: numbers by (head,
+    distance) that join the scores, the last of a head for all further distances."""
     which, more = ("", ()) if heads is None else ("_heads", heads)
+    turn = (lib.ptr(ocos), lib.ptr(osin))
+    if dist_bias is not None:
+        which, turn = "_biased", ()
+        more = (heads or (0, 1.0, o.stride(0))) + (lib.ptr(dist_bias), dist_bias.shape[1] - 1)
     sfx = lib.suffix(m.dtype)
     q_stride = m.qkv_width if q_stride is None else q_stride
     if m.window_tile and USE_WINDOW_MMA:
@@ -438,7 +498,7 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
                         lib.ptr(gate), lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos),
                         lib.ptr(table), lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width,
                         m.nh, m.nkvh, m.dh, m.dv, splits, window, m.keep_first, m.scale, m.softcap, m.chunk,
-                        lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin), *more):
+                        lib.ptr(sinks), *turn, *more):
             return
     tiles = ctx.tiles(m.general_tile)
     # slices of the visited keys so that a few sequences still fill the GPU: a function of the batch's shape alone (a
@@ -450,4 +510,4 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
     lib.call(f"tb_attention_window{which}_{sfx}", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v), lib.ptr(gate),
              lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos), lib.ptr(table),
              lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width, m.nh, m.nkvh, m.dh, m.dv,
-             splits, window, m.keep_first, m.scale, m.softcap, m.chunk, lib.ptr(sinks), lib.ptr(ocos), lib.ptr(osin), *more)
+             splits, window, m.keep_first, m.scale, m.softcap, m.chunk, lib.ptr(sinks), *turn, *more)

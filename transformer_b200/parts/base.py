@@ -33,6 +33,8 @@ InputFilter   changes what a part reads, row by row or along time: ``forward(ctx
 Joint         rewrites the whole residual stream between two runs of the model: ``begin(ctx, x)`` right after
               the embedding (to keep what it needs of it), ``forward(ctx, x, pending)`` before the run that
               names it (``pending`` is what the run before left to be added; it returns what is still pending).
+ResidualGate  multiplies a part's result before it joins the stream, by a function of what that part reads:
+              ``forward(ctx, y)`` gives the gate's pre-activation [nt, d] and its bias; the sum applies them.
 ============  ===================================================================================
 
 All parts declare their parameters with :meth:`Part.parameters` (name -> shape, role, init) and
@@ -113,6 +115,32 @@ class NormedDelta:
 
 
 @dataclass
+class GatedDelta:
+    """A part's output that passes a bias and a gate of its own on its way into the stream, element by element:
+    x += (delta + delta_bias) * sigmoid(gate + gate_bias); each of the three but ``delta`` may be missing.  A norm that
+    sets ``takes_gated_delta`` does the sum in its own kernel; for any other the block adds it to the stream first."""
+    delta: torch.Tensor                            # [nt, d]
+    delta_bias: Optional[torch.Tensor] = None      # float [d]
+    gate: Optional[torch.Tensor] = None            # [nt, d]
+    gate_bias: Optional[torch.Tensor] = None       # float [d]
+
+    def moved(self, of: Callable) -> "GatedDelta":
+        """The same left by another run of an equal layer: ``of`` maps a layer's own tensor to the other layer's."""
+        return GatedDelta(self.delta, of(self.delta_bias), self.gate, of(self.gate_bias))
+
+
+@dataclass
+class DepthSum:
+    """The stream is still to be replaced by a weighted sum over the depth of the model: with ``pending`` added first,
+    X = x (which is kept as the last of ``terms`` rows of ``history``), x <- sum_j weights[j] history[j].  Norms with
+    ``takes_gated_delta`` do all of it in their own kernel."""
+    pending: Any               # a tensor, a GatedDelta or None
+    history: torch.Tensor      # float [>= terms, nt, d]; the first terms - 1 are filled
+    weights: torch.Tensor      # float [terms]
+    terms: int
+
+
+@dataclass
 class StreamRows:
     """Nothing is left to be added to the stream, and the stream's rows, rounded to the activation type, already lie in
     ``rows``: left by a block whose last kernel norms the stream itself, for a block that reads it as it is."""
@@ -177,6 +205,7 @@ class Norm(Part):
     takes_weighted_rows = False
     takes_normed_delta = False
     takes_pair_delta = False
+    takes_gated_delta = False  # a GatedDelta or a DepthSum
     can_warm = False           # forward takes ``warm=``: a weight of the next part to fetch into L2 meanwhile
     tails: tuple = ()          # kinds of NormTail that forward(..., tail=) computes along the way
     renew_tails: tuple = ()    # the same for renew(..., tail=)
@@ -192,6 +221,8 @@ class Norm(Part):
 
 class Mixer(Part):
     rows_width: Optional[int] = None    # the width of the rows that forward_rows leaves for the output product
+    has_out_bias = False                # ``out_bias``, float [d], is still to be added to what forward writes: the block
+    out_bias: Optional[torch.Tensor] = None      # does that where it adds the result to the stream (``takes_out_bias``)
 
     def cache_need(self) -> Optional[CacheNeed]:
         return None
@@ -233,6 +264,12 @@ class Joint(Part):
         """Called once per step with the embedding output ``x`` (float [nt, d]), before any layer runs."""
 
     def forward(self, ctx, x, pending):
+        raise NotImplementedError
+
+
+class ResidualGate(Part):
+    def forward(self, ctx, y) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+        """The gate's pre-activation for the rows ``y`` that the gated part reads, and a bias to be added to it."""
         raise NotImplementedError
 
 
@@ -301,4 +338,5 @@ FEED_FORWARDS = Registry("feed-forward")
 POSITIONS = Registry("position encoding")
 INPUT_FILTERS = Registry("input filter")
 JOINTS = Registry("joint")
+RESIDUAL_GATES = Registry("residual gate")
 ARRANGEMENTS = Registry("block arrangement")     # kind -> class(LayerSpec, dtype, device); see parts/block.py

@@ -4,7 +4,7 @@
 
     x += mixer(norm_m(x));   x += feed_forward(norm_f(x))
 
-The residual stream ``x`` is float.  A part writes its contribution ``delta``; the sum into ``x``
+A layer may have no feed-forward, and either result may pass a gate first (see :class:`Layer`).  The residual stream ``x`` is float.  A part writes its contribution ``delta``; the sum into ``x``
 is fused into the NEXT norm (of this block or the following one, or the final norm), so a block
 takes the pending delta of the block before it and returns its own.
 
@@ -17,27 +17,42 @@ return value is what this block leaves.  A block that wants its sums done at onc
 """
 from __future__ import annotations
 
-from .base import ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, NormedDelta, PairDelta, StreamRows, WeightedRows
+from .base import (ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, RESIDUAL_GATES, DepthSum, GatedDelta, NormedDelta,
+                   PairDelta, StreamRows, WeightedRows)
 from .spec import PartSpec
 
 
 def build_layer(spec, dtype, device):
     """The block of one LayerSpec, by its arrangement."""
-    return ARRANGEMENTS.get(spec.arrangement)(spec, dtype, device)
+    layer = ARRANGEMENTS.get(spec.arrangement)(spec, dtype, device)
+    if layer.mixer.has_out_bias and not getattr(layer, "takes_out_bias", False):
+        raise ValueError(f"a mixer of kind {spec.mixer.kind!r} whose output bias the block adds does not go with the "
+                         f"arrangement {spec.arrangement!r}")
+    return layer
 
 
 @ARRANGEMENTS.register("pre_norm")
 class Layer:
-    """The parts of one LayerSpec, built, in the pre-norm arrangement."""
+    """The parts of one LayerSpec, built, in the pre-norm arrangement.  A layer may have no feed-forward.
+    ``LayerSpec.extra`` may name a "mixer_residual_gate" and a "feed_forward_residual_gate": the part's result is then
+    multiplied by the gate, a function of what the part reads, where it joins the stream (:class:`GatedDelta`)."""
+    takes_out_bias = True
 
     def __init__(self, spec, dtype, device):
-        if spec.mixer_norm is None or spec.feed_forward_norm is None:
+        if spec.mixer_norm is None or (spec.feed_forward is not None and spec.feed_forward_norm is None):
             raise ValueError("the pre_norm arrangement needs a norm before the mixer and one before the feed-forward")
+        extra = dict(spec.extra)
         self.spec = spec
         self.mixer_norm = NORMS.build(spec.mixer_norm, dtype, device)
         self.mixer = MIXERS.build(spec.mixer, dtype, device)
-        self.feed_forward_norm = NORMS.build(spec.feed_forward_norm, dtype, device)
-        self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, dtype, device)
+        self.feed_forward = self.feed_forward_norm = None
+        if spec.feed_forward is not None:
+            self.feed_forward_norm = NORMS.build(spec.feed_forward_norm, dtype, device)
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, dtype, device)
+        self.gates = {n: RESIDUAL_GATES.build(extra[n + "_residual_gate"], dtype, device) for n in ("mixer", "feed_forward")
+                      if n + "_residual_gate" in extra}
+        if "feed_forward" in self.gates and self.feed_forward is None:
+            raise ValueError("a gate on the feed-forward's result needs a feed-forward")
 
     @property
     def graph_safe(self) -> bool:
@@ -48,28 +63,48 @@ class Layer:
         return all(p.launches_only for p in self.parts().values())
 
     def parts(self):
-        return {"mixer_norm": self.mixer_norm, "mixer": self.mixer,
-                "feed_forward_norm": self.feed_forward_norm, "feed_forward": self.feed_forward}
+        out = {"mixer_norm": self.mixer_norm, "mixer": self.mixer}
+        if self.feed_forward is not None:
+            out.update({"feed_forward_norm": self.feed_forward_norm, "feed_forward": self.feed_forward})
+        out.update({n + "_residual_gate": g for n, g in self.gates.items()})
+        return out
+
+    def _gate(self, which, ctx, y):
+        """(pre-activation, bias) of the gate of this part, read from the rows the part reads."""
+        return self.gates[which].forward(ctx, y) if which in self.gates else (None, None)
 
     def forward(self, ctx, x, pending, cache_view, state):
         """x: float [nt, d]; pending: the previous block's delta or None.  Returns this block's
-        pending delta (the feed-forward's output)."""
+        pending delta (its last part's output)."""
         nt, d = x.shape
         x1 = ctx.scratch("block.x1", (nt, d), ctx.dtype)
         delta = ctx.scratch("block.delta", (nt, d), ctx.dtype)
         pending = resolve(pending, self.mixer_norm, delta, x=x, ctx=ctx)
         self._norm(self.mixer_norm, self.mixer, ctx, x, pending, x1)
+        gate, gate_bias = self._gate("mixer", ctx, x1)
         self.mixer.forward(ctx, x1, delta, cache_view, state)
+        result = delta
+        if gate is not None or self.mixer.out_bias is not None:
+            result = GatedDelta(delta, self.mixer.out_bias, gate, gate_bias)
+        if self.feed_forward is None:
+            return result
+        result = resolve(result, self.feed_forward_norm, delta, x=x, ctx=ctx)
         tail = self.feed_forward.norm_tail(ctx, nt)
         if tail is not None and tail.kind in self.feed_forward_norm.tails:
             # the feed-forward's first small step rides along with the norm before it
-            self.feed_forward_norm.forward(ctx, x, delta, None, x1, tail=tail)
-            lazy = self.feed_forward.forward(ctx, x1, delta, tail=tail)
+            self.feed_forward_norm.forward(ctx, x, result, None, x1, tail=tail)
         else:
-            self._norm(self.feed_forward_norm, self.feed_forward, ctx, x, delta, x1)
-            lazy = self.feed_forward.forward(ctx, x1, delta)
-        return delta if lazy is None else lazy
-
+            tail = None
+            self._norm(self.feed_forward_norm, self.feed_forward, ctx, x, result, x1)
+        gate, gate_bias = self._gate("feed_forward", ctx, x1)
+        lazy = self.feed_forward.forward(ctx, x1, delta) if tail is None else \
+            self.feed_forward.forward(ctx, x1, delta, tail=tail)
+        if gate is None:
+            return delta if lazy is None else lazy
+        if lazy is not None:
+            from .feed_forward import sum_weighted_rows
+            sum_weighted_rows(lazy, delta)
+        return GatedDelta(delta, None, gate, gate_bias)
 
     @staticmethod
     def _norm(norm, then, ctx, x, delta, y) -> None:
@@ -225,7 +260,7 @@ class ParallelLayer:
         h2 = ctx.scratch("block.x2", (nt, d), ctx.dtype) if self.feed_forward is not None else None
         out_m = ctx.scratch("block.delta", (nt, d), ctx.dtype)
         out_f = ctx.scratch("block.delta2", (nt, d), ctx.dtype) if self.feed_forward is not None else None
-        if isinstance(pending, (NormedDelta, WeightedRows)):
+        if isinstance(pending, (NormedDelta, WeightedRows, GatedDelta, DepthSum)):
             pending = resolve(pending, None, out_m, x=x, ctx=ctx)
         if self._fused:
             pair_add_rmsnorm(ctx.dtype, x, pending, None, self.mixer_norm.weights["weight"], h1,
@@ -320,6 +355,10 @@ def add_pending(ctx, x, pending) -> None:
         from .norm import pair_add_rmsnorm
         pair_add_rmsnorm(ctx.dtype, x, pending, None, None, None, None, None, 0.0)
         return
+    if isinstance(pending, (GatedDelta, DepthSum)):
+        from .norm import stream_step
+        stream_step(ctx.dtype, x, pending, None, None, None)
+        return
     if isinstance(pending, WeightedRows):
         from .feed_forward import sum_weighted_rows
         into = ctx.scratch("block.delta", tuple(x.shape), ctx.dtype)
@@ -338,6 +377,13 @@ def resolve(pending, norm, into, x=None, ctx=None):
             return pending
         if x is None or ctx is None:
             raise ValueError("a normed delta can only be resolved with the stream at hand")
+        add_pending(ctx, x, pending)
+        return None
+    if isinstance(pending, (GatedDelta, DepthSum)):
+        if getattr(norm, "takes_gated_delta", False):
+            return pending
+        if x is None or ctx is None:
+            raise ValueError("a gated output can only be resolved with the stream at hand")
         add_pending(ctx, x, pending)
         return None
     if isinstance(pending, PairDelta):

@@ -11,8 +11,10 @@ from __future__ import annotations
 import torch
 
 from ..csrc import lib
-from .base import EMBEDDINGS, HEADS, Embedding, Head, ParamDecl, StateNeed
+from .base import EMBEDDINGS, HEADS, NORMS, Embedding, Head, ParamDecl, StateNeed
 from .linear import matmul_nt
+from .norm import TanhNorm
+from .spec import PartSpec
 
 
 @EMBEDDINGS.register("lookup")
@@ -68,6 +70,37 @@ class BigramLookup(Embedding):
                  lib.ptr(ctx.tok_pos), lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), lib.ptr(state),
                  lib.ptr(self.weights["table"]), lib.ptr(self.weights["pairs"]), lib.ptr(x), x.shape[0], self.width,
                  self.scale, self.buckets, self.mul_prev, self.mul_cur)
+
+
+@EMBEDDINGS.register("positional_lookup")
+class PositionalLookup(Embedding):
+    """params: vocab, width, positions; optional: scale (default 1), norm (a PartSpec of kind "tanh_norm").
+
+        x[i] = table[tok_i] * scale + positions[pos_i]        (pos_i: the token's position in its sequence)
+
+    in float; with ``norm`` (parameters "norm.*") the stream starts with the norm of that, in the same kernel."""
+    graph_safe = True
+
+    def __init__(self, params, dtype, device):
+        super().__init__(params, dtype, device)
+        self.vocab, self.width, self.count = int(params["vocab"]), int(params["width"]), int(params["positions"])
+        self.scale = float(params.get("scale", 1.0))
+        norm = params.get("norm")
+        self.norm = NORMS.build(norm, dtype, device) if isinstance(norm, PartSpec) else None
+        if self.norm is not None and not isinstance(self.norm, TanhNorm):
+            raise ValueError(f"the embedding's own norm is one without statistics ('tanh_norm'), not {norm.kind!r}")
+
+    def parameters(self):
+        decl = {"table": ParamDecl((self.vocab, self.width)), "positions": ParamDecl((self.count, self.width))}
+        if self.norm is not None:
+            decl.update({"norm." + n: d for n, d in self.norm.parameters().items()})
+        return decl
+
+    def forward(self, ctx, x) -> None:
+        w = self.weights
+        lib.call("tb_embed_learned_" + lib.suffix(self.dtype), lib.ptr(ctx.tok_ids), lib.ptr(ctx.tok_pos),
+                 lib.ptr(w["table"]), lib.ptr(w["positions"]), lib.ptr(x), x.shape[0], self.width, self.scale,
+                 lib.ptr(w.get("norm.alpha")), lib.ptr(w.get("norm.weight")), lib.ptr(w.get("norm.bias")))
 
 
 @HEADS.register("linear")

@@ -1,9 +1,10 @@
 """RMSNorm fused with the residual sum (models/llama/common/src/compute.rs:207,275,362); a layer norm (mean taken
-off, weight and bias, an optional multiplier per channel) with the same fusions; and no norm at all."""
+off, weight and bias, an optional multiplier per channel) with the same fusions; a norm without statistics, tanh of the
+scaled stream; and no norm at all."""
 from __future__ import annotations
 
 from ..csrc import lib
-from .base import NORMS, Norm, NormedDelta, PairDelta, ParamDecl, WeightedRows
+from .base import NORMS, DepthSum, GatedDelta, Norm, NormedDelta, PairDelta, ParamDecl, WeightedRows
 
 
 @NORMS.register("rmsnorm")
@@ -153,6 +154,28 @@ class LayerNorm(Norm):
                  lib.ptr(y), y.shape[0], self.width, *pick)
 
 
+@NORMS.register("tanh_norm")
+class TanhNorm(Norm):
+    """params: width.  y = tanh(alpha v) * weight + bias with a learned number alpha: no mean, no variance, so every entry
+    is on its own and one kernel over the entries does all that stands between a part's output and the next part's
+    input: bias and gate of the output (:class:`GatedDelta`), the float sum, a weighted sum over the model's depth
+    (:class:`DepthSum`) and the norm.  csrc/stream_step.cu."""
+    graph_safe = True
+    launches_only = True
+    takes_gated_delta = True
+
+    def __init__(self, params, dtype, device):
+        super().__init__(params, dtype, device)
+        self.width = int(params["width"])
+
+    def parameters(self):
+        return {"weight": ParamDecl((self.width,), "norm", "ones"), "bias": ParamDecl((self.width,), "norm", "normal"),
+                "alpha": ParamDecl((), "norm", "ones")}
+
+    def forward(self, ctx, x, delta, rows, y) -> None:
+        stream_step(self.dtype, x, delta, rows, self.weights, y)
+
+
 @NORMS.register("none")
 class NoNorm(Norm):
     """params: width.  No norm at all, for blocks whose parts read the residual stream as it is: the pending
@@ -254,6 +277,23 @@ def post_add_layernorm(dtype, x, delta, post, rows, weight, bias, eps, center, y
              1 if center else 0, lib.ptr(y), n_out, x.shape[1])
     if tail is not None and y is not None:
         _route(lib.suffix(dtype), y, tail, n_out, x.shape[1])
+
+
+def stream_step(dtype, x, pending, rows, norm, y) -> None:
+    """x[rows] <- what ``pending`` (a tensor, a :class:`GatedDelta`, a :class:`DepthSum` or None) makes of it, written back
+    when ``rows`` is None; then y = tanh(alpha x) * weight + bias with ``norm`` = {"alpha", "weight", "bias"}, or the
+    stream itself without one.  ``y`` None: only the stream."""
+    history = weights = None
+    terms = 0
+    if isinstance(pending, DepthSum):
+        history, weights, terms, pending = pending.history, pending.weights, pending.terms, pending.pending
+    g = pending if isinstance(pending, GatedDelta) else GatedDelta(pending)
+    norm = norm or {}
+    lib.call("tb_stream_step_" + lib.suffix(dtype), lib.ptr(x), lib.ptr(g.delta), lib.ptr(g.delta_bias), lib.ptr(g.gate),
+             0 if g.gate is None else g.gate.stride(0), lib.ptr(g.gate_bias), lib.ptr(history),
+             0 if history is None else history.stride(0), lib.ptr(weights), terms, lib.ptr(rows), lib.ptr(norm.get("alpha")),
+             lib.ptr(norm.get("weight")), lib.ptr(norm.get("bias")), lib.ptr(y),
+             x.shape[0] if rows is None else rows.shape[0], x.shape[1])
 
 
 def pair_add_rmsnorm(dtype, x, pending, rows, w1, y1, w2, y2, eps) -> None:

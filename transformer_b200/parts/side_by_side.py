@@ -25,6 +25,10 @@ class SideBySide(Mixer):
             if m.rows_width is None:
                 raise ValueError(f"a mixer of kind {params[n].kind!r} does not leave its rows to another part's product")
         self.tile_sizes = sorted({int(t) for m in self.sides.values() for t in getattr(m, "tile_sizes", ())})
+        biased = [n for n, m in self.sides.items() if m.has_out_bias]
+        if len(biased) > 1:
+            raise ValueError("only one of two mixers side by side may have a bias on its output")
+        self.has_out_bias = bool(biased)
         self.cached = self._the_one("cache", lambda m: m.cache_need())
         self.stateful = self._the_one("state", lambda m: m.state_need())
 
@@ -53,6 +57,8 @@ class SideBySide(Mixer):
             m.bind({k: tensors[f"{n}.{k}"] for k in m.parameters()})
             outs.append(m.weights.pop("wo"))
             self.weights.update({f"{n}.{k}": t for k, t in m.weights.items()})
+            if m.has_out_bias:
+                self.out_bias = m.out_bias
         self.weights["wo"] = torch.cat(outs, dim=1).contiguous()
 
     def cache_need(self):

@@ -12,7 +12,8 @@ which architecture it came from.
   (weights shared, each run with a cache entry of its own unless told otherwise) or let a run read
   the cache that another run wrote (``cache_of``).
 * ``ModelSpec.joints`` are parts that rewrite the whole residual stream between two runs (a projection that
-  mixes the embedding output back in, ...); a :class:`RunEntry` names the one that runs right before it.
+  mixes the embedding output back in, ...); a :class:`RunEntry` names the one that runs right before it, and
+  ``ModelSpec.last_joint`` the one that runs behind the last run, before the model's last norm.
 """
 from __future__ import annotations
 
@@ -62,10 +63,13 @@ class ModelSpec:
     head: PartSpec
     stop_tokens: Tuple[int, ...] = ()
     joints: Tuple[PartSpec, ...] = ()
+    last_joint: Optional[int] = None      # index into joints of the part that rewrites the stream behind the last run
 
     def validate(self) -> None:
         if not self.layers:
             raise ValueError("a model needs at least one layer")
+        if self.last_joint is not None and not (0 <= self.last_joint < len(self.joints)):
+            raise ValueError(f"the last joint is number {self.last_joint}, but there are {len(self.joints)}")
         for i, e in enumerate(self.order):
             if not (0 <= e.layer < len(self.layers)):
                 raise ValueError(f"run entry {i} names layer {e.layer}, but there are {len(self.layers)}")
