@@ -6,6 +6,7 @@
     python bench.py --design zufadra [--sizes s,m]      the Zufadra design beside a dense Llama at equal sizes
     python bench.py --design fugavik [--sizes s,m]      the Fugavik design beside Zufadra, Dumalix and Llama-MoE
     python bench.py --design fofapel [--sizes s,m]      the Fofapel design beside Fugavik, Zufadra and Llama-MoE
+    python bench.py --design tubazen [--sizes s,m]      the Tubazen design beside Fofapel and Zufadra
 
 The default run has the layer sizes of the LLaMA-MoE-3.5B (4/16) shape (32 layers, width 4096,
 32/32 heads of 128, 16 experts top-4 of width 688, vocabulary 32000, context 4096) with random
@@ -276,6 +277,34 @@ def fofapel_shapes(size):
     return fofapel, fugavik_shapes(size)[0], zufadra_shapes(size)[0], design_shapes(size)[1]
 
 
+def tubazen_shapes(size):
+    """(Tubazen config, Fofapel config, Zufadra config) for a named size.  The Tubazen layers alternate between the two
+    mixers side by side and the gated linear attention, each with the dense feed-forward.  Fofapel with dense feed-forwards
+    everywhere (two mixers side by side, a linear memory with a decay per key channel, windowed attention, a norm kernel per
+    part) is the closest model for everything but the delta rule; Zufadra has the delta rule, attention over all earlier
+    positions with a gate per entry (its window is the context) and the same dense feed-forward."""
+    d, L, H, G, dim, rank, ff = {
+        "s": (1024, 8, 8, 2, 128, 64, 2816),
+        "m": (2048, 8, 16, 4, 128, 128, 5632),
+    }[size]
+    par = {"left": {"heads": H, "kv_heads": G, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_max": 1000, "bias_rows": 64,
+                    "q_temp": {"coef": 0.1, "every": 1024}},
+           "right": {"heads": H, "dim": dim, "decay_rank": rank}, "left_scale": 0.9, "right_scale": 0.6}
+    gla = {"heads": H, "dim": dim, "vdim": dim, "tau": 8.0, "decay_rank": rank}
+    mlp = {"kind": "dense", "ff": ff}
+    tubazen = {"architecture": "Tubazen", "vocab": 32000, "width": d, "norm": {"eps": 1e-6}, "logit_scale": 1.5,
+               "max_positions": 8192,
+               "layers": [{"type": "parallel" if i % 2 == 0 else "gla", "mixer": par if i % 2 == 0 else gla, "mlp": mlp}
+                          for i in range(L)]}
+    fofapel = fofapel_shapes(size)[0]
+    fofapel["layers"] = [dict(l, mlp=mlp, mixer=dict(l["mixer"], left=dict(l["mixer"]["left"], mask={"size": 8192})))
+                         for l in fofapel["layers"]]
+    zufadra = zufadra_shapes(size)[0]
+    zufadra["layers"] = [l if l["type"] != "attention" else dict(l, mixer=dict(l["mixer"], mask={"size": 8192, "keep_first": 4}))
+                         for l in zufadra["layers"]]
+    return tubazen, fofapel, zufadra
+
+
 def bench_design(args):
     """Prefill and decode throughput of another design beside the closest existing model of equal sizes, and the
     device time of every kernel family in one eager step of each (CUDA events around each launch).  One JSON line."""
@@ -291,7 +320,8 @@ def bench_design(args):
                      "zufadra": (("zufadra", "llama_dense"), zufadra_shapes),
                      "dumalix": (("dumalix", "zufadra_attention", "salepel"), dumalix_shapes),
                      "fugavik": (("fugavik", "zufadra", "dumalix", "llama_moe"), fugavik_shapes),
-                     "fofapel": (("fofapel", "fugavik", "zufadra", "llama_moe"), fofapel_shapes)}[args.design]
+                     "fofapel": (("fofapel", "fugavik", "zufadra", "llama_moe"), fofapel_shapes),
+                     "tubazen": (("tubazen", "fofapel_dense", "zufadra_full"), tubazen_shapes)}[args.design]
     out = {"metric": f"prefill and decode tok/s, {names[0]} beside {' and '.join(names[1:])} at equal sizes", "unit": "tokens/s",
            "dtype": "bf16" if args.dtype == "bfloat16" else "fp32", "data": "synthetic: random weights, random token ids",
            "peaks": pk, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx0, "steps": K, "warmup": W,
@@ -387,7 +417,7 @@ def main():
                     help="layer sizes: the benchmark's (default) or another shape BASELINE.json names")
     ap.add_argument("--prompt-max", type=int, default=0, help="longest prompt drawn (default: the shape's own)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS)
-    ap.add_argument("--design", default=None, choices=["salepel", "zufadra", "dumalix", "fugavik", "fofapel"],
+    ap.add_argument("--design", default=None, choices=["salepel", "zufadra", "dumalix", "fugavik", "fofapel", "tubazen"],
                     help="instead of the default workload: this design beside the closest existing model at equal "
                          "sizes (prefill of --prefill-tokens, decode at --batch; sizes from --sizes)")
     ap.add_argument("--sizes", default="s,m", help="with --design: which of the named sizes (s, m)")

@@ -3,6 +3,7 @@ their own (experiments, tests): every parameter a part declares becomes one file
 
     embedding.<param>, head.<param> (``head.weight`` is absent when the head is tied), final_norm.<param>,
     layers.<i>.<part of the block>.<param>       (pre_norm: mixer_norm | mixer | feed_forward_norm | feed_forward)
+    joints.<i>.<param>
 """
 from __future__ import annotations
 
@@ -10,7 +11,7 @@ from typing import List
 
 import torch
 
-from ..parts.base import EMBEDDINGS, HEADS, NORMS
+from ..parts.base import EMBEDDINGS, HEADS, JOINTS, NORMS
 from ..parts.block import build_layer
 from ..parts.spec import ModelSpec
 from ..weights.plan import TensorRule, single
@@ -30,6 +31,8 @@ def plan_from_spec(spec: ModelSpec) -> List[TensorRule]:
     for i, ls in enumerate(spec.layers):
         for pname, part in build_layer(ls, torch.bfloat16, cpu).parts().items():
             declare(("layers", i, pname), f"layers.{i}.{pname}", part)
+    for i, j in enumerate(spec.joints):
+        declare(("joints", i), f"joints.{i}", JOINTS.build(j, torch.bfloat16, cpu))
     declare(("final_norm",), "final_norm", NORMS.build(spec.final_norm, torch.bfloat16, cpu))
     tied = bool(spec.head.get().get("tied", False))
     declare(("head",), "head", HEADS.build(spec.head, torch.bfloat16, cpu),

@@ -110,13 +110,14 @@ __global__ void __launch_bounds__(128) stream_step_kernel(const StreamStepArgs a
 
 template <typename T>
 static int stream_step_launch(const StreamStepArgs& a, cudaStream_t s) {
-    if (!a.x || a.n_out < 0 || a.d <= 0 || a.terms < 0) return TB_ERR_ARG;
+    if (a.n_out < 0 || a.d <= 0 || a.terms < 0) return TB_ERR_ARG;
+    if (a.n_out == 0) return 0;
+    if (!a.x) return TB_ERR_ARG;
     if (a.terms > 0 && (!a.history || !a.c || a.hstride < a.d)) return TB_ERR_ARG;
     if ((a.gate || a.delta_b) && !a.delta) return TB_ERR_ARG;
     if (a.gate ? a.ldg < a.d : a.gate_b != nullptr) return TB_ERR_ARG;
     if ((a.w != nullptr) != (a.alpha != nullptr) || (a.w != nullptr) != (a.b != nullptr)) return TB_ERR_ARG;
     if (a.rows && !a.y) return TB_ERR_ARG;
-    if (a.n_out == 0) return 0;
     const uintptr_t all = (uintptr_t)a.x | (uintptr_t)a.delta | (uintptr_t)a.delta_b | (uintptr_t)a.gate | (uintptr_t)a.gate_b |
                           (uintptr_t)a.history | (uintptr_t)a.w | (uintptr_t)a.b | (uintptr_t)a.y;
     const bool vec = a.d % 8 == 0 && a.ldg % 8 == 0 && a.hstride % 4 == 0 && (all & 15) == 0;
@@ -160,9 +161,9 @@ template <typename T>
 static int embed_learned_launch(const int* tokens, const int* positions, const void* table, const void* ptable, float* x,
                                 int nt, int d, float scale, const float* alpha, const float* w, const float* b,
                                 cudaStream_t s) {
+    if (nt == 0) return 0;
     if (nt < 0 || d <= 0 || !tokens || !positions || !table || !ptable || !x) return TB_ERR_ARG;
     if ((w != nullptr) != (alpha != nullptr) || (w != nullptr) != (b != nullptr)) return TB_ERR_ARG;
-    if (nt == 0) return 0;
     const bool vec = d % 8 == 0 &&
                      (((uintptr_t)table | (uintptr_t)ptable | (uintptr_t)x | (uintptr_t)w | (uintptr_t)b) & 15) == 0;
     const long long n = (long long)nt * (d / (vec ? 8 : 1)), blocks = (n + 127) / 128;
