@@ -26,7 +26,6 @@
 #define SD_UNIT_EPS 1e-6f
 #define SD_RATE 0.60653065971263342f    // e^(-1/2)
 
-constexpr int SD_SCAN = 128;            // threads of a scan block
 constexpr int SD_STEP = 512;            // threads of a step block
 
 __host__ __device__ inline int sd_record(int dim) { return 5 * dm_rows(dim) + 4; }
@@ -132,13 +131,13 @@ struct SplitDeltaScanArgs {
     int nt, H, dim;
 };
 
-// RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): SD_SCAN / SPLIT * C columns a
+// RPT rows of C columns per thread, SPLIT lanes per column (SPLIT * RPT = dm_rows(dim)): THREADS / SPLIT * C columns a
 // block.  The records of TOK tokens at a time are one bulk copy to shared memory, STAGES - 1 stages ahead.
-template <int RPT, int SPLIT, int C, int TOK, int STAGES>
-__global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDeltaScanArgs a) {
+template <int RPT, int SPLIT, int C, int THREADS, int TOK, int STAGES>
+__global__ void __launch_bounds__(THREADS) split_delta_scan_kernel(const SplitDeltaScanArgs a) {
     pdl_sync();
     constexpr int DP = RPT * SPLIT;
-    constexpr int COLS = SD_SCAN / SPLIT * C;
+    constexpr int COLS = THREADS / SPLIT * C;
     constexpr int ROW = 5 * DP + 4;                     // a record
     constexpr int NV = TOK * C;
     static_assert(NV % SPLIT == 0, "every lane ends with as many sums");
@@ -177,7 +176,7 @@ __global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDe
             bulk_load(smem_u32(to), rec + (size_t)ts * ROW, bytes, bar0 + 8u * (q % STAGES));
         }
         // tokens behind the last: nothing is written, nothing fades, nothing is read (so that a stage has no branches)
-        for (int idx = n * ROW + tid; idx < TOK * ROW; idx += SD_SCAN) {
+        for (int idx = n * ROW + tid; idx < TOK * ROW; idx += THREADS) {
             const int e = idx % ROW;
             to[idx] = e >= 2 * DP && e < 3 * DP ? 1.f : 0.f;
         }
@@ -207,17 +206,19 @@ __global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDe
                 p[c][0].f.x = p[c][0].f.y = p[c][1].f.x = p[c][1].f.y = d[c].f.x = d[c].f.y = 0.f;
             }
             // the sums over the old state
+            union Four { float4 f; F2 p[2]; };
+            Four u[RPT / 4];
 #pragma unroll
             for (int i4 = 0; i4 < RPT / 4; ++i4) {
                 const int ch = i4 * SPLIT + part;
-                union { float4 f; F2 p[2]; } rw, u;
+                Four rw;
                 rw.f = reinterpret_cast<const float4*>(row)[ch];
-                u.f = reinterpret_cast<const float4*>(row + DP)[ch];
+                u[i4].f = reinterpret_cast<const float4*>(row + DP)[ch];
 #pragma unroll
                 for (int c = 0; c < C; ++c)
 #pragma unroll
                     for (int q = 0; q < 2; ++q) {
-                        p[c][q] = fma2(s[c][i4 * 2 + q], u.p[q], p[c][q]);
+                        p[c][q] = fma2(s[c][i4 * 2 + q], u[i4].p[q], p[c][q]);
                         d[c] = fma2(s[c][i4 * 2 + q], rw.p[q], d[c]);
                     }
             }
@@ -239,8 +240,7 @@ __global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDe
 #pragma unroll
             for (int i4 = 0; i4 < RPT / 4; ++i4) {
                 const int ch = i4 * SPLIT + part;
-                union { float4 f; F2 p[2]; } u, w, na;
-                u.f = reinterpret_cast<const float4*>(row + DP)[ch];
+                Four w, na;
                 w.f = reinterpret_cast<const float4*>(row + 2 * DP)[ch];
                 na.f = reinterpret_cast<const float4*>(row + 3 * DP)[ch];
 #pragma unroll
@@ -248,7 +248,7 @@ __global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDe
 #pragma unroll
                     for (int q = 0; q < 2; ++q) {
                         F2& si = s[c][i4 * 2 + q];
-                        si = fma2(na.p[q], p[c][0], fma2(si, w.p[q], mul2(u.p[q], v[c])));
+                        si = fma2(na.p[q], p[c][0], fma2(si, w.p[q], mul2(u[i4].p[q], v[c])));
                     }
             }
         }
@@ -282,22 +282,22 @@ __global__ void __launch_bounds__(SD_SCAN) split_delta_scan_kernel(const SplitDe
         }
 }
 
-template <int RPT, int SPLIT, int C, int TOK, int STAGES>
+template <int RPT, int SPLIT, int C, int THREADS, int TOK, int STAGES>
 static int split_delta_scan_go(const SplitDeltaScanArgs& a, int B, bool early, cudaStream_t s) {
-    constexpr int COLS = SD_SCAN / SPLIT * C;
+    constexpr int COLS = THREADS / SPLIT * C;
     constexpr size_t smem = (size_t)STAGES * TOK * (5 * RPT * SPLIT + 4) * sizeof(float);
     static_assert(smem <= 220 * 1024, "the stages fit an SM");
     static bool configured = false;
     if (smem > 48 * 1024 && !configured) {
-        cudaError_t e = cudaFuncSetAttribute(split_delta_scan_kernel<RPT, SPLIT, C, TOK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(split_delta_scan_kernel<RPT, SPLIT, C, THREADS, TOK, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(B, a.H, (a.dim + COLS - 1) / COLS);
     if (early)
-        TB_LAUNCH((split_delta_scan_kernel<RPT, SPLIT, C, TOK, STAGES>), grid, SD_SCAN, smem, s, a);
+        TB_LAUNCH((split_delta_scan_kernel<RPT, SPLIT, C, THREADS, TOK, STAGES>), grid, THREADS, smem, s, a);
     else        // prompts: the blocks run for the whole sequence and want an SM each (see tb_launch_plain)
-        tb_launch_plain(split_delta_scan_kernel<RPT, SPLIT, C, TOK, STAGES>, grid, dim3(SD_SCAN), smem, s, a);
+        tb_launch_plain(split_delta_scan_kernel<RPT, SPLIT, C, THREADS, TOK, STAGES>, grid, dim3(THREADS), smem, s, a);
     return tb_last_error();
 }
 
@@ -308,15 +308,23 @@ static int split_delta_scan_launch(SplitDeltaScanArgs a, int B, cudaStream_t s) 
     a.error = tc_error_ptr();
     if (!a.error) return tb_last_error();
     const bool early = a.nt <= 2 * B;
-    const bool many = (long long)B * a.H * a.dim >= 128 * 32;
+    // Few columns of state in the batch: small pieces per thread, so that as many warps as there are keep the chain of a
+    // token short (one prompt of 2,048 tokens: 16 heads of 128 387 us with 4 rows of 2 columns and 256 threads, 492 with 16
+    // rows of 1 and 128; 8 heads of 128 324 us with 4 of 2 and 128 threads; 32 heads of 64 304 us with 4 of 1, 360 with 8 of
+    // 1).  Enough of them to fill the GPU: larger pieces, which read a record's entry for more columns (eight prompts of 512
+    // tokens: 16 heads of 128 371 us with 16 rows of 2, 707 with 4 of 2; 32 heads of 64 190 us with 8 of 4, 401 with 8 of 1).
+    const long long columns = (long long)B * a.H * a.dim;
+    const bool many = columns >= 128 * 32;
     switch (dm_rows(a.dim)) {
-        case 16: return split_delta_scan_go<4, 4, 1, 8, 4>(a, B, early, s);
-        case 32: return split_delta_scan_go<4, 8, 1, 8, 4>(a, B, early, s);
+        case 16: return split_delta_scan_go<4, 4, 1, 128, 8, 4>(a, B, early, s);
+        case 32: return split_delta_scan_go<4, 8, 1, 128, 8, 4>(a, B, early, s);
         case 64:
-            return many ? split_delta_scan_go<8, 8, 2, 8, 4>(a, B, early, s) : split_delta_scan_go<8, 8, 1, 8, 4>(a, B, early, s);
+            return many ? split_delta_scan_go<8, 8, 4, 64, 8, 4>(a, B, early, s) : split_delta_scan_go<4, 16, 1, 128, 16, 3>(a, B, early, s);
         case 128:
-            return many ? split_delta_scan_go<16, 8, 2, 8, 4>(a, B, early, s) : split_delta_scan_go<16, 8, 1, 8, 4>(a, B, early, s);
-        default: return split_delta_scan_go<16, 16, 1, 16, 2>(a, B, early, s);
+            return many              ? split_delta_scan_go<16, 8, 2, 128, 8, 4>(a, B, early, s)
+                   : columns > 1024 ? split_delta_scan_go<4, 32, 2, 256, 16, 3>(a, B, early, s)
+                                    : split_delta_scan_go<4, 32, 2, 128, 16, 3>(a, B, early, s);
+        default: return split_delta_scan_go<16, 16, 1, 128, 16, 2>(a, B, early, s);
     }
 }
 

@@ -120,6 +120,8 @@ class Engine:
         for i, layer in enumerate(self.layers):
             for pname, part in layer.parts().items():
                 part.bind({n: weights[("layers", i, pname, n)] for n in part.parameters()})
+            if hasattr(layer, "bound"):
+                layer.bound()
         self.final_norm.bind({n: weights[("final_norm", n)] for n in self.final_norm.parameters()})
         for i, joint in enumerate(self.joints):
             joint.bind({n: weights[("joints", i, n)] for n in joint.parameters()})

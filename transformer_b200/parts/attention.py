@@ -176,6 +176,8 @@ class Attention(Mixer):
             self.qkv_width = (self.proj_rows + 7) // 8 * 8
         if self.extended and not self.prepared:
             self.rows_width = self.nh * self.dv
+            if not self.keyed:
+                self.in_weight, self.in_width = "wqkv", self.qkv_width
         self.q_mult = None
         if self.query_temp is not None:
             coef, every = float(self.query_temp[0]), int(self.query_temp[1])
@@ -311,13 +313,15 @@ class Attention(Mixer):
                              sinks=w.get("sink"), ocos=vcos, osin=vsin)
         matmul_nt(o, w["wo"], out)
 
-    def _window_rows(self, ctx, x1, rows, cache) -> None:
+    def _window_rows(self, ctx, x1, rows, cache, z=None) -> None:
         """The step with the further mechanisms up to its output product: see the head of this file."""
         nt = x1.shape[0]
         sfx = lib.suffix(self.dtype)
         w = self.weights
-        z = ctx.scratch("attn.qkv", (nt, self.qkv_width), self.dtype)        # q | k | v | gate
-        matmul_nt(x1, w["wqkv"], z)
+        if z is None:
+            z = ctx.scratch("attn.qkv", (nt, self.qkv_width), self.dtype)    # q | k | v | gate
+            matmul_nt(x1, w["wqkv"], z)
+        ldz = z.stride(0)
         table = ctx.page_table(cache)
         cos = sin = None
         half = 0
@@ -327,22 +331,23 @@ class Attention(Mixer):
         which, first = "", ()
         if self.bias or self.q_mult is not None:
             which, first = "biased_", (lib.ptr(w.get("bqkv")), lib.ptr(self.q_mult))
-        lib.call("tb_qknorm_rope_cache_" + which + sfx, lib.ptr(z), self.qkv_width, *first, lib.ptr(w.get("q_norm")),
+        lib.call("tb_qknorm_rope_cache_" + which + sfx, lib.ptr(z), ldz, *first, lib.ptr(w.get("q_norm")),
                  lib.ptr(w.get("k_norm")), self.eps, lib.ptr(ctx.tok_seq), lib.ptr(ctx.tok_pos), lib.ptr(table),
                  ctx.max_pages, lib.ptr(cos), lib.ptr(sin), lib.ptr(kc), lib.ptr(vc), nt, self.nh, self.nkvh, self.dh,
                  self.dv, self.rdims, half)
         gate = z[:, (self.nh + self.nkvh) * self.dh + self.nkvh * self.dv:] if self.gate else None
         window = self.window if self.window else 1 << 30
         plain = self.out_scale == 1.0 and rows.stride(0) == self.nh * self.dv
-        run_window_attention(ctx, self, z, rows, gate, cache, table, nt, window, sinks=w.get("sink") if self.sink else None,
+        run_window_attention(ctx, self, z, rows, gate, cache, table, nt, window, q_stride=ldz,
+                             sinks=w.get("sink") if self.sink else None,
                              heads=None if plain else (0, self.out_scale, rows.stride(0)), dist_bias=w.get("rel"))
 
-    def forward_rows(self, ctx, x1, rows, cache, state) -> None:
+    def forward_rows(self, ctx, x1, rows, cache, state, z=None) -> None:
         """The heads' outputs, gated and scaled."""
         if self.rows_width is None:
             raise NotImplementedError("attention of this family does not leave its rows to another part's product")
         if not self.keyed:
-            self._window_rows(ctx, x1, rows, cache)
+            self._window_rows(ctx, x1, rows, cache, z)
             return
         nt = x1.shape[0]
         w = self.weights
@@ -363,10 +368,10 @@ class Attention(Mixer):
                              q_stride=self.nh * self.dh, sinks=w.get("sink"),
                              heads=(1 if self.head_gate else 0, self.out_scale, rows.stride(0)))
 
-    def forward(self, ctx, x1, out, cache, state) -> None:
+    def forward(self, ctx, x1, out, cache, state, z=None) -> None:
         if self.rows_width is not None:
             rows = ctx.scratch("attn.o", (x1.shape[0], self.rows_width), self.dtype)
-            self.forward_rows(ctx, x1, rows, cache, state)
+            self.forward_rows(ctx, x1, rows, cache, state, z)
             matmul_nt(rows, self.weights["wo"], out)
             return
         if self.prepared:
@@ -486,6 +491,7 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
         more = (heads or (0, 1.0, o.stride(0))) + (lib.ptr(dist_bias), dist_bias.shape[1] - 1)
     sfx = lib.suffix(m.dtype)
     q_stride = m.qkv_width if q_stride is None else q_stride
+    g_stride = m.qkv_width if gate is None else gate.stride(0)
     if m.window_tile and USE_WINDOW_MMA:
         # bfloat16: the tensor-core kernel, for prompts and decoding alike.  Slices of the visited pages so that a few
         # sequences still fill the GPU: a function of the batch's shape alone (a captured graph keeps it)
@@ -496,7 +502,7 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
         partial = ctx.scratch("attn.partial", (nt, m.nh, splits, m.dv + 2), torch.float32) if splits > 1 else None
         if lib.try_call(f"tb_attention_window_mma{which}_bf16", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v),
                         lib.ptr(gate), lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos),
-                        lib.ptr(table), lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width,
+                        lib.ptr(table), lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, g_stride,
                         m.nh, m.nkvh, m.dh, m.dv, splits, window, m.keep_first, m.scale, m.softcap, m.chunk,
                         lib.ptr(sinks), *turn, *more):
             return
@@ -509,5 +515,5 @@ def run_window_attention(ctx, m, z, o, gate, cache, table, nt, window, q_stride=
     partial = ctx.scratch("attn.partial", (nt, m.nh, splits, m.dv + 2), torch.float32) if splits > 1 else None
     lib.call(f"tb_attention_window{which}_{sfx}", lib.ptr(z), lib.ptr(o), lib.ptr(cache.k), lib.ptr(cache.v), lib.ptr(gate),
              lib.ptr(tiles.seq), lib.ptr(tiles.t0), lib.ptr(tiles.nq), lib.ptr(ctx.tok_pos), lib.ptr(table),
-             lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, m.qkv_width, m.nh, m.nkvh, m.dh, m.dv,
+             lib.ptr(partial), tiles.count, nt, ctx.max_pages, q_stride, g_stride, m.nh, m.nkvh, m.dh, m.dv,
              splits, window, m.keep_first, m.scale, m.softcap, m.chunk, lib.ptr(sinks), *turn, *more)

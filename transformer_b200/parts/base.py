@@ -221,6 +221,9 @@ class Norm(Part):
 
 class Mixer(Part):
     rows_width: Optional[int] = None    # the width of the rows that forward_rows leaves for the output product
+    in_weight: Optional[str] = None     # name of the weight [in_width, width] of a first product z = x1 weight^T that whoever
+    in_width: int = 0                   # calls the mixer may do together with others that read x1: ``forward`` and
+                                        # ``forward_rows`` then take the rows (a view with a pitch) as ``z=``
     has_out_bias = False                # ``out_bias``, float [d], is still to be added to what forward writes: the block
     out_bias: Optional[torch.Tensor] = None      # does that where it adds the result to the stream (``takes_out_bias``)
 
@@ -268,7 +271,10 @@ class Joint(Part):
 
 
 class ResidualGate(Part):
-    def forward(self, ctx, y) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    product: Optional[str] = None       # name of the weight [d, width] if the pre-activation is y weight^T: the block may
+                                        # do that product together with another one and hand its rows over as ``z=``
+
+    def forward(self, ctx, y, z=None) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         """The gate's pre-activation for the rows ``y`` that the gated part reads, and a bias to be added to it."""
         raise NotImplementedError
 

@@ -19,6 +19,7 @@ from __future__ import annotations
 
 from .base import (ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, RESIDUAL_GATES, DepthSum, GatedDelta, NormedDelta,
                    PairDelta, StreamRows, WeightedRows)
+from .linear import matmul_nt, stack_products
 from .spec import PartSpec
 
 
@@ -51,6 +52,7 @@ class Layer:
             self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, dtype, device)
         self.gates = {n: RESIDUAL_GATES.build(extra[n + "_residual_gate"], dtype, device) for n in ("mixer", "feed_forward")
                       if n + "_residual_gate" in extra}
+        self._joined = None     # where the gate's columns begin in the mixer's first product, if they are one product
         if "feed_forward" in self.gates and self.feed_forward is None:
             raise ValueError("a gate on the feed-forward's result needs a feed-forward")
 
@@ -69,6 +71,17 @@ class Layer:
         out.update({n + "_residual_gate": g for n, g in self.gates.items()})
         return out
 
+    def bound(self) -> None:
+        """Called when all parts have their weights.  The mixer's first product and its gate's read the same rows: where
+        the mixer lets its own be done for it, the two become one."""
+        gate = self.gates.get("mixer")
+        self._joined = None
+        if gate is None or not self.mixer.in_weight or not gate.product:
+            return
+        w = self.mixer.weights
+        w[self.mixer.in_weight], starts = stack_products([w[self.mixer.in_weight], gate.weights.pop(gate.product)])
+        self._joined = starts[1]
+
     def _gate(self, which, ctx, y):
         """(pre-activation, bias) of the gate of this part, read from the rows the part reads."""
         return self.gates[which].forward(ctx, y) if which in self.gates else (None, None)
@@ -81,8 +94,15 @@ class Layer:
         delta = ctx.scratch("block.delta", (nt, d), ctx.dtype)
         pending = resolve(pending, self.mixer_norm, delta, x=x, ctx=ctx)
         self._norm(self.mixer_norm, self.mixer, ctx, x, pending, x1)
-        gate, gate_bias = self._gate("mixer", ctx, x1)
-        self.mixer.forward(ctx, x1, delta, cache_view, state)
+        if self._joined is not None:
+            w = self.mixer.weights[self.mixer.in_weight]
+            z = ctx.scratch("block.z", (nt, w.shape[0]), ctx.dtype)
+            matmul_nt(x1, w, z)
+            gate, gate_bias = self.gates["mixer"].forward(ctx, x1, z=z[:, self._joined:])
+            self.mixer.forward(ctx, x1, delta, cache_view, state, z=z[:, :self.mixer.in_width])
+        else:
+            gate, gate_bias = self._gate("mixer", ctx, x1)
+            self.mixer.forward(ctx, x1, delta, cache_view, state)
         result = delta
         if gate is not None or self.mixer.out_bias is not None:
             result = GatedDelta(delta, self.mixer.out_bias, gate, gate_bias)

@@ -55,11 +55,11 @@ class GatedLinear(Mixer):
             raise ValueError(f"the gated linear attention's kernels take heads of up to 256 key entries, got {self.dim}")
         self.hk, self.hv = self.H * self.dim, self.H * self.vdim
         self.rows_width = self.hv
-        self.z_width = 2 * self.hk + 2 * self.hv
+        self.in_weight, self.in_width = "win", 2 * self.hk + 2 * self.hv
 
     def parameters(self):
         return {
-            "win": ParamDecl((self.z_width, self.d)),             # rows: q heads, k heads, v heads, output gate
+            "win": ParamDecl((self.in_width, self.d)),             # rows: q heads, k heads, v heads, output gate
             "a1": ParamDecl((self.rank, self.d)),
             "a2": ParamDecl((self.hk, self.rank)),
             "a2_bias": ParamDecl((self.hk,), "norm", "normal"),
@@ -76,17 +76,19 @@ class GatedLinear(Mixer):
     def state_need(self):
         return StateNeed(((self.hk * self.vdim + 3) // 4 * 4,), torch.float32)
 
-    def forward_rows(self, ctx, x1, rows, cache, state) -> None:
+    def forward_rows(self, ctx, x1, rows, cache, state, z=None) -> None:
         nt, H = x1.shape[0], self.H
         sfx = lib.suffix(self.dtype)
         w = self.weights
         pitch = state.stride(0)
-        z = ctx.scratch("gla.z", (nt, self.z_width), self.dtype)
-        matmul_nt(x1, w["win"], z)
+        if z is None:
+            z = ctx.scratch("gla.z", (nt, self.in_width), self.dtype)
+            matmul_nt(x1, w["win"], z)
+        ldz = z.stride(0)
         a = ctx.scratch("gla.a", (nt, self.rank), torch.float32)
         matmul_nt(x1, w["a1"], a)                                           # float out on both paths
         if ctx.decode and USE_STEP and lib.try_call(
-                "tb_gated_linear_step_" + sfx, lib.ptr(z), self.z_width, lib.ptr(a), self.rank, lib.ptr(w["a2"]),
+                "tb_gated_linear_step_" + sfx, lib.ptr(z), ldz, lib.ptr(a), self.rank, lib.ptr(w["a2"]),
                 lib.ptr(w["a2_bias"]), lib.ptr(w["norm"]), lib.ptr(state), pitch, lib.ptr(rows), rows.stride(0),
                 lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, H, self.dim, self.vdim, self.rank, 1.0 / self.tau,
                 self.dim ** -0.5, self.eps):
@@ -97,16 +99,16 @@ class GatedLinear(Mixer):
         matmul_nt(split, w["a2_split"], pre)                                # float out
         size = lib.gated_linear_record_size(self.dim, self.vdim)
         rec = ctx.scratch("gla.rec", (H, nt, size), torch.float32)
-        lib.call("tb_gated_linear_prep_" + sfx, lib.ptr(z), self.z_width, lib.ptr(pre), lib.ptr(w["a2_bias"]), lib.ptr(rec),
+        lib.call("tb_gated_linear_prep_" + sfx, lib.ptr(z), ldz, lib.ptr(pre), lib.ptr(w["a2_bias"]), lib.ptr(rec),
                  nt, H, self.dim, self.vdim, size, 1.0 / self.tau, self.dim ** -0.5)
         o = ctx.scratch("gla.o", (nt, self.hv), torch.float32)
         lib.call("tb_decay_scan_rect", lib.ptr(rec), lib.ptr(state), pitch, lib.ptr(o), lib.ptr(ctx.seq_start),
                  lib.ptr(ctx.slots), nt, ctx.B, H, self.dim, self.vdim)
         gate = z[:, 2 * self.hk + self.hv:]
-        lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(gate), self.z_width, lib.ptr(w["norm"]), lib.ptr(rows), nt, H,
+        lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(gate), ldz, lib.ptr(w["norm"]), lib.ptr(rows), nt, H,
                  self.vdim, self.eps, 1, rows.stride(0))
 
-    def forward(self, ctx, x1, out, cache, state) -> None:
+    def forward(self, ctx, x1, out, cache, state, z=None) -> None:
         rows = ctx.scratch("gla.y", (x1.shape[0], self.hv), self.dtype)
-        self.forward_rows(ctx, x1, rows, cache, state)
+        self.forward_rows(ctx, x1, rows, cache, state, z)
         matmul_nt(rows, self.weights["wo"], out)

@@ -128,6 +128,18 @@ def matmul_nt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, w_is_weigh
         torch.mm(a, w.t(), out=out)
 
 
+def stack_products(weights):
+    """Weights [n_i, width] of products with the same rows as ONE weight, and where each one's columns begin in the
+    product: at multiples of eight (rows of zeros between them), so that each part of a row is aligned like a row."""
+    pieces, starts, at = [], [], 0
+    for w in weights:
+        pad = (w.shape[0] + 7) // 8 * 8 - w.shape[0]
+        starts.append(at)
+        pieces += [w] if not pad else [w, w.new_zeros((pad, w.shape[1]))]
+        at += w.shape[0] + pad
+    return torch.cat(pieces, dim=0).contiguous(), starts
+
+
 def grouped_matmul(a, w, out, *, a_rows=None, group_offsets=None, groups=1, swiglu=False, max_group_rows=0,
                    scratch=None, w_is_weight: bool = True, glu=None) -> None:
     """out[m] = a[a_rows[m] or m] . w[g(m)]^T over rows sorted by group; with swiglu, w[g] holds gate rows

@@ -41,6 +41,7 @@ class SplitDelta(Mixer):
         if self.dim > 256:
             raise ValueError(f"the split delta rule's kernels take heads of up to 256 entries, got {self.dim}")
         self.rows_width = self.hd = self.H * self.dim
+        self.in_weight, self.in_width = "win", 4 * self.hd
 
     def parameters(self):
         return {
@@ -62,18 +63,20 @@ class SplitDelta(Mixer):
     def state_need(self):
         return StateNeed(((self.hd * self.dim + 3) // 4 * 4,), torch.float32)
 
-    def forward_rows(self, ctx, x1, rows, cache, state) -> None:
+    def forward_rows(self, ctx, x1, rows, cache, state, z=None) -> None:
         nt, H, hd = x1.shape[0], self.H, self.hd
         sfx = lib.suffix(self.dtype)
         w = self.weights
         pitch = state.stride(0)
-        z = ctx.scratch("sdelta.z", (nt, 4 * hd), self.dtype)
-        matmul_nt(x1, w["win"], z)
+        if z is None:
+            z = ctx.scratch("sdelta.z", (nt, 4 * hd), self.dtype)
+            matmul_nt(x1, w["win"], z)
+        ldz = z.stride(0)
         wide = hd + self.rank
         az = ctx.scratch("sdelta.a", (nt, wide), torch.float32)
         matmul_nt(x1, w["wa"], az)                                          # float out on both paths
         if ctx.decode and USE_STEP and lib.try_call(
-                "tb_split_delta_step_" + sfx, lib.ptr(z), 4 * hd, lib.ptr(az), wide, lib.ptr(w["ba"]), lib.ptr(w["w2"]),
+                "tb_split_delta_step_" + sfx, lib.ptr(z), ldz, lib.ptr(az), wide, lib.ptr(w["ba"]), lib.ptr(w["w2"]),
                 lib.ptr(w["w0"]), lib.ptr(w["norm"]), self.eps, lib.ptr(state), pitch, lib.ptr(rows), rows.stride(0),
                 lib.ptr(ctx.seq_start), lib.ptr(ctx.slots), nt, ctx.B, H, self.dim, self.rank):
             return
@@ -82,15 +85,15 @@ class SplitDelta(Mixer):
         pre = ctx.scratch("sdelta.pre", (nt, hd), torch.float32)
         matmul_nt(th, w["w2_split"], pre)                                   # float out
         rec = ctx.scratch("sdelta.rec", (H, nt, lib.split_delta_record_size(self.dim)), torch.float32)
-        lib.call("tb_split_delta_prep_" + sfx, lib.ptr(z), 4 * hd, lib.ptr(az), wide, lib.ptr(w["ba"]), lib.ptr(pre),
+        lib.call("tb_split_delta_prep_" + sfx, lib.ptr(z), ldz, lib.ptr(az), wide, lib.ptr(w["ba"]), lib.ptr(pre),
                  lib.ptr(w["w0"]), lib.ptr(rec), nt, H, self.dim)
         o = ctx.scratch("sdelta.o", (nt, hd), torch.float32)
         lib.call("tb_split_delta_scan", lib.ptr(rec), lib.ptr(state), pitch, lib.ptr(o), lib.ptr(ctx.seq_start),
                  lib.ptr(ctx.slots), nt, ctx.B, H, self.dim)
-        lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(z[:, 3 * hd:]), 4 * hd, lib.ptr(w["norm"]), lib.ptr(rows), nt, H,
+        lib.call("tb_mlstm_out_" + sfx, lib.ptr(o), lib.ptr(z[:, 3 * hd:]), ldz, lib.ptr(w["norm"]), lib.ptr(rows), nt, H,
                  self.dim, self.eps, 0, rows.stride(0))
 
-    def forward(self, ctx, x1, out, cache, state) -> None:
+    def forward(self, ctx, x1, out, cache, state, z=None) -> None:
         rows = ctx.scratch("sdelta.y", (x1.shape[0], self.hd), self.dtype)
-        self.forward_rows(ctx, x1, rows, cache, state)
+        self.forward_rows(ctx, x1, rows, cache, state, z)
         matmul_nt(rows, self.weights["wo"], out)

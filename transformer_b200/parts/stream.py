@@ -112,6 +112,7 @@ class SigmoidGate(ResidualGate):
     """params: width.  sigmoid(weight y + bias); the sigmoid and the bias are the sum's business."""
     graph_safe = True
     launches_only = True
+    product = "weight"
 
     def __init__(self, params, dtype, device):
         super().__init__(params, dtype, device)
@@ -120,7 +121,8 @@ class SigmoidGate(ResidualGate):
     def parameters(self):
         return {"weight": ParamDecl((self.width, self.width)), "bias": ParamDecl((self.width,), "norm", "normal")}
 
-    def forward(self, ctx, y):
-        gate = ctx.scratch("block.gate", (y.shape[0], self.width), self.dtype)
-        matmul_nt(y, self.weights["weight"], gate)
-        return gate, self.weights["bias"]
+    def forward(self, ctx, y, z=None):
+        if z is None:
+            z = ctx.scratch("block.gate", (y.shape[0], self.width), self.dtype)
+            matmul_nt(y, self.weights["weight"], z)
+        return z, self.weights["bias"]
