@@ -27,6 +27,11 @@ from .context import StepContext, Workspace, weak_callback
 from .tape import LayerTape, moves, run_tensors
 
 
+# From this many tokens on the device has more to do than the interpreter: a sum over the depth then rides in the norm of
+# the layer behind it, and the layer is run from Python; below, it is a pass of its own, and equal layers are replayed.
+FUSE_DEPTH_ROWS = 1024
+
+
 class StepError(ValueError):
     pass
 
@@ -371,10 +376,13 @@ class Engine:
                 pending = self.joints[entry.joint].forward(ctx, x, pending)
             kind = self._run_kind[r] if taping else None
             if kind is not None and isinstance(pending, DepthSum) and not ctx.decode:
-                # many tokens: the sum is done here, so that the layer's launches name no tensor of the joint's (layers
-                # of equal parts are then replayed with their own tensors put in)
-                add_pending(ctx, x, pending)
-                pending = None
+                if nt >= FUSE_DEPTH_ROWS:
+                    kind = None
+                else:
+                    # the sum is done here, so that the layer's launches name no tensor of the joint's (layers of equal
+                    # parts are then replayed with their own tensors put in)
+                    add_pending(ctx, x, pending)
+                    pending = None
             if kind is None:
                 pending = layer.forward(ctx, x, pending, self.cache.view(r), self.cache.state_of(r))
                 continue
