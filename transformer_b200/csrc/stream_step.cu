@@ -63,23 +63,8 @@ __global__ void __launch_bounds__(128) stream_step_kernel(const StreamStepArgs a
     if (!mine) return;
     const int r = a.rows ? a.rows[i] : i;
     const size_t at = (size_t)r * a.d + col;
-    float v[V], s[V];
+    float v[V];
     ss_loadf<V>(a.x + at, v);
-    // the sum over the depth first: its reads then wait together with those of the delta
-    const int last = a.terms - 1;
-#pragma unroll
-    for (int e = 0; e < V; ++e) s[e] = 0.f;
-    if (a.terms > 0) {
-        const float* hp = a.history + at;
-#pragma unroll 4
-        for (int j = 0; j < last; ++j, hp += a.hstride) {
-            float h[V];
-            ss_loadf<V>(hp, h);
-            const float cj = a.c[j];
-#pragma unroll
-            for (int e = 0; e < V; ++e) s[e] += cj * h[e];
-        }
-    }
     if (a.delta) {
         float u[V];
         ss_load<T, V>(static_cast<const T*>(a.delta) + at, u);
@@ -95,7 +80,20 @@ __global__ void __launch_bounds__(128) stream_step_kernel(const StreamStepArgs a
         for (int e = 0; e < V; ++e) v[e] += u[e];
     }
     if (a.terms > 0) {
+        const int last = a.terms - 1;
         if (!a.rows) ss_store<float, V>(a.history + (size_t)last * a.hstride + at, v);
+        float s[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] = 0.f;
+        const float* hp = a.history + at;
+#pragma unroll 4
+        for (int j = 0; j < last; ++j, hp += a.hstride) {
+            float h[V];
+            ss_loadf<V>(hp, h);
+            const float cj = a.c[j];
+#pragma unroll
+            for (int e = 0; e < V; ++e) s[e] += cj * h[e];
+        }
         const float cl = a.c[last];
 #pragma unroll
         for (int e = 0; e < V; ++e) v[e] = s[e] + cl * v[e];
